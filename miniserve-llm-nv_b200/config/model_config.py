@@ -949,3 +949,147 @@ class BafavikConfig:
         loop = None if self.loop is None else dict(start=self.loop[0], stop=self.loop[1], times=self.loop[2])
         return dict(architecture=self.architecture, vocab=self.vocab, width=self.width, norm=dict(eps=self.eps),
                     residual_mult=self.residual_mult, logit_scale=self.logit_scale, embedding=embedding, loop=loop, layers=layers)
+
+
+# --------------------------------------------------------------------------- Venarax
+
+
+def _window_or_none(data: Mapping[str, Any], where: str) -> Any:
+    """``mask.size`` of a mixer whose tokens see themselves and the ``size - 1`` tokens before them (no ``mask``: every token)."""
+    if data.get("mask") is None:
+        return None
+    return _integer(_section(data, "mask", where), "size")
+
+
+@dataclass(frozen=True)
+class WindowedLatentAttentionConfig:
+    """Latent attention with an interleaved rotation of a part that all heads share, a sliding window and a gate per entry."""
+
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot: RotationConfig
+    window: Any
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], where: str) -> "WindowedLatentAttentionConfig":
+        latent = LatentAttentionConfig.from_dict(data, where)
+        if latent.rot.scaling is not None:
+            raise UnsupportedModelError(f"UNSUPPORTED_MODEL_CONFIGURATION: {where}rot.scaling is not implemented for this design")
+        return cls(heads=latent.heads, dim=latent.dim, rot_dim=latent.rot_dim, vdim=latent.vdim, kv_rank=latent.kv_rank,
+                   scale=latent.scale, rot=latent.rot, window=_window_or_none(data, where))
+
+    def to_dict(self) -> dict[str, Any]:
+        out = dict(heads=self.heads, dim=self.dim, rot_dim=self.rot_dim, vdim=self.vdim, kv_rank=self.kv_rank, scale=self.scale,
+                   rot=dict(base=self.rot.base, dims=self.rot.dims))
+        if self.window is not None:
+            out["mask"] = dict(size=self.window)
+        return out
+
+
+@dataclass(frozen=True)
+class SinkAttentionConfig:
+    """Grouped-query attention without rotation: queries and keys normed over the whole projection, a learned sink per head and a
+    temperature of the queries that grows with the position (``temperature``: (coef, every), or None)."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    temperature: Any
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], where: str) -> "SinkAttentionConfig":
+        temperature = None
+        if data.get("q_temp") is not None:
+            raw = _section(data, "q_temp", where)
+            coef = _number(raw, "coef")
+            if not math.isfinite(coef):
+                raise ValueError(f"{where}q_temp.coef must be finite, got {coef}")
+            temperature = (coef, _positive(raw, "every", where + "q_temp."))
+        config = cls(heads=_integer(data, "heads"), kv_heads=_integer(data, "kv_heads"), dim=_integer(data, "dim"),
+                     vdim=_integer(data, "vdim"), scale=_positive(data, "scale", where), temperature=temperature)
+        if config.heads % config.kv_heads:
+            raise ValueError(f"{where}heads {config.heads} is not a multiple of kv_heads {config.kv_heads}")
+        return config
+
+    def to_dict(self) -> dict[str, Any]:
+        out: dict[str, Any] = dict(heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, scale=self.scale)
+        if self.temperature is not None:
+            out["q_temp"] = dict(coef=self.temperature[0], every=self.temperature[1])
+        return out
+
+
+@dataclass(frozen=True)
+class ClampedFeedForwardConfig:
+    ff: int
+    limit: float
+
+
+@dataclass(frozen=True)
+class VenaraxLayerConfig:
+    type: str       # "latent_attention" or "attention"
+    mixer: Any
+    mlp: Any        # ClampedFeedForwardConfig or None
+
+
+@dataclass(frozen=True)
+class VenaraxConfig:
+    """The Venarax decoder: ``config.json`` holds ``architecture``, ``vocab``, ``width``, ``norm.eps``, ``loop`` (``start``, ``stop``,
+    ``times``: those layers run that often in a row, or null) and ``layers``, a list whose entries give each layer's mixer ``type``
+    (``latent_attention`` or ``attention``), the mixer's sizes and constants (``mixer``) and its feed-forward (``mlp`` with ``kind``
+    "dense", ``ff`` and ``limit``, or null).  Every size and constant is read."""
+
+    vocab: int
+    width: int
+    eps: float
+    loop: Any       # None or (start, stop, times)
+    layers: tuple
+    architecture: str = "Venarax"
+
+    MIXERS = {"latent_attention": WindowedLatentAttentionConfig.from_dict, "attention": SinkAttentionConfig.from_dict}
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any]) -> "VenaraxConfig":
+        if data.get("architecture") != "Venarax":
+            raise UnsupportedModelError(f"UNSUPPORTED_MODEL_CONFIGURATION: expected architecture 'Venarax', got {data.get('architecture')!r}")
+        raw_layers = data.get("layers")
+        if not isinstance(raw_layers, (list, tuple)) or not raw_layers:
+            raise ValueError("layers must be a non-empty list in the model config")
+        layers = []
+        for index, raw in enumerate(raw_layers):
+            where = f"layers[{index}]."
+            if not isinstance(raw, Mapping):
+                raise ValueError(f"layers[{index}] must be an object")
+            kind = raw.get("type")
+            if kind not in cls.MIXERS:
+                raise UnsupportedModelError(f"UNSUPPORTED_MODEL_CONFIGURATION: {where}type {kind!r} is not implemented "
+                                            f"({', '.join(cls.MIXERS)})")
+            mixer = cls.MIXERS[kind](_section(raw, "mixer", where), where + "mixer.")
+            mlp = None
+            if raw.get("mlp") is not None:
+                data_mlp = _section(raw, "mlp", where)
+                if data_mlp.get("kind") != "dense":
+                    raise UnsupportedModelError(f"UNSUPPORTED_MODEL_CONFIGURATION: {where}mlp.kind {data_mlp.get('kind')!r} is not implemented (dense)")
+                mlp = ClampedFeedForwardConfig(_integer(data_mlp, "ff"), _positive(data_mlp, "limit", where + "mlp."))
+            layers.append(VenaraxLayerConfig(kind, mixer, mlp))
+        loop = None
+        if data.get("loop") is not None:
+            raw = _section(data, "loop", "")
+            loop = (_count(raw, "start", 0), _integer(raw, "stop"), _integer(raw, "times"))
+            if not loop[0] < loop[1] <= len(layers):
+                raise ValueError(f"loop: layers {loop[0]} .. {loop[1]} - 1 are not a run of the model's {len(layers)} layers")
+        return cls(vocab=_integer(data, "vocab"), width=_integer(data, "width"), eps=_positive(_section(data, "norm", ""), "eps", "norm."),
+                   loop=loop, layers=tuple(layers))
+
+    def to_dict(self) -> dict[str, Any]:
+        """The ``config.json`` content that reads back as this configuration."""
+        layers = [dict(type=layer.type, mixer=layer.mixer.to_dict(),
+                       mlp=None if layer.mlp is None else dict(kind="dense", ff=layer.mlp.ff, limit=layer.mlp.limit))
+                  for layer in self.layers]
+        loop = None if self.loop is None else dict(start=self.loop[0], stop=self.loop[1], times=self.loop[2])
+        return dict(architecture=self.architecture, vocab=self.vocab, width=self.width, norm=dict(eps=self.eps), loop=loop, layers=layers)

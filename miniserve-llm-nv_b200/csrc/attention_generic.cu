@@ -18,7 +18,7 @@
 //
 // Three more options.  Value heads may have another size dv than query and key heads (d): the pools then differ in
 // their last dimension and the output has dv numbers per head.  `sink`: the softmax's denominator gets one more term
-// exp(0), a key of score 0 without a value, p_j = exp(s_j) / (1 + sum exp(s_j)).  `gate`: the head's output is
+// exp(0), a key of score 0 without a value, p_j = exp(s_j) / (1 + sum exp(s_j)), or exp(sink_scores[head]), a score per query head.  `gate`: the head's output is
 // multiplied by sigmoid(gate[token, head]) as it is stored.
 #include "common.cuh"
 
@@ -71,7 +71,8 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, const T*
                                                const int* __restrict__ positions, int page_size, int n_q, int n_kv,
                                                int d, float scale, int window, float softcap,
                                                const float* __restrict__ bias_slopes, T* __restrict__ out, int dv,
-                                               int sink, const T* __restrict__ gate, int gate_ld, int chunk, int n_v) {
+                                               int sink, const float* __restrict__ sink_scores, const T* __restrict__ gate, int gate_ld,
+                                               int chunk, int n_v) {
   grid_dependency_wait();
   grid_dependency_launch();
   extern __shared__ float smem[];
@@ -144,11 +145,12 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, const T*
     if (c < dv) part_acc[warp * dv + c] = acc[i];
   }
   __syncthreads();
-  float m_all = sink ? 0.f : -INFINITY;               // the sink is a key of score 0
+  const float sink_score = sink && sink_scores ? sink_scores[head] : 0.f;
+  float m_all = sink ? sink_score : -INFINITY;        // the sink is a key of score 0, or of the head's own score
   for (int w = 0; w < kAttnWarps; ++w) m_all = fmaxf(m_all, part_m[w]);
   float l_all = 0.f;
   for (int w = 0; w < kAttnWarps; ++w) l_all += part_m[w] == -INFINITY ? 0.f : part_l[w] * expf(part_m[w] - m_all);
-  if (sink) l_all += expf(-m_all);
+  if (sink) l_all += expf(sink_score - m_all);
   float factor = 1.f / l_all;
   if (gate) factor /= 1.f + expf(-to_float(gate[(size_t)token * gate_ld + head]));
   T* out_row = out + ((size_t)token * n_q + head) * dv;
@@ -169,7 +171,7 @@ using namespace ms;
 // The keys of a token are positions max(0, pos - window + 1) .. pos of its own request
 // (window <= 0: no window); they must already be in the pool.  softcap <= 0: no soft cap; bias_slopes
 // [n_q] float32 or null.  dv: the size of a value head (value pool [pages, n_kv, page_size, dv], out [n_tokens, n_q, dv]);
-// sink != 0: one more term exp(0) in the softmax's denominator; gate (null: none): logits of the model's element type,
+// sink != 0: one more term exp(0), or exp(sink_scores[head]) (float32 [n_q], not null), in the softmax's denominator; gate (null: none): logits of the model's element type,
 // gate[token * gate_ld + head], whose sigmoid multiplies the head's output.  chunk > 0: a token sees only the keys of its own
 // chunk of `chunk` positions (position p: keys p - p % chunk .. p).  n_v: the value pool holds that many heads, [pages, n_v,
 // page_size, dv] (a divisor of n_kv; key head g reads value head g % n_v: key heads that share values).
@@ -177,7 +179,8 @@ MS_EXPORT int ms_paged_attention_generic(const void* q, int dtype, const void* k
                                          const int* block_tables, int table_stride, const int* request_of_token,
                                          const int* positions, int page_size, int n_q, int n_kv, int d, float scale,
                                          int window, float softcap, const float* bias_slopes, void* out, int n_tokens,
-                                         int dv, int sink, const void* gate, int gate_ld, int chunk, int n_v, cudaStream_t stream) {
+                                         int dv, int sink, const float* sink_scores, const void* gate, int gate_ld, int chunk, int n_v,
+                                         cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   MS_REQUIRE(d > 0 && d <= 32 * kMaxLanesPerThread, "paged_attention: head size %d outside 1..%d", d,
              32 * kMaxLanesPerThread);
@@ -193,13 +196,13 @@ MS_EXPORT int ms_paged_attention_generic(const void* q, int dtype, const void* k
   if (dtype == MS_F32) {
     ms::launch(paged_attention_generic_kernel<float>, grid, kAttnWarps * 32, smem, stream, 
         (const float*)q, (const float*)k_pool, (const float*)v_pool, block_tables, table_stride, request_of_token,
-        positions, page_size, n_q, n_kv, d, scale, window, softcap, bias_slopes, (float*)out, dv, sink,
+        positions, page_size, n_q, n_kv, d, scale, window, softcap, bias_slopes, (float*)out, dv, sink, sink_scores,
         (const float*)gate, gate_ld, chunk, n_v);
   } else if (dtype == MS_BF16) {
     ms::launch(paged_attention_generic_kernel<__nv_bfloat16>, grid, kAttnWarps * 32, smem, stream, 
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, block_tables,
         table_stride, request_of_token, positions, page_size, n_q, n_kv, d, scale, window, softcap, bias_slopes,
-        (__nv_bfloat16*)out, dv, sink, (const __nv_bfloat16*)gate, gate_ld, chunk, n_v);
+        (__nv_bfloat16*)out, dv, sink, sink_scores, (const __nv_bfloat16*)gate, gate_ld, chunk, n_v);
   } else {
     MS_FAIL("paged_attention: unknown element type code %d", dtype);
   }

@@ -17,11 +17,16 @@ constexpr int kLatWarps = 4;
 constexpr int kLatMaxLanes = 32;   // value lanes per thread: R up to 1024
 
 // Rotation of element c of a vector of `rot` entries whose first `dims` are rotated: entry j < dims / 2 is paired
-// with entry j + dims / 2; the table holds (cos, sin) of the token for each pair (already times the magnitude).
+// with entry j + dims / 2 (interleaved: entry 2j with entry 2j + 1); the table holds (cos, sin) of the token for each pair (already times the magnitude).
 template <typename T>
-__device__ __forceinline__ float rotated(const T* src, int c, int dims, const float2* table) {
+__device__ __forceinline__ float rotated(const T* src, int c, int dims, const float2* table, int interleaved) {
   const float v = to_float(src[c]);
   if (c >= dims) return v;
+  if (interleaved) {
+    const float2 cs = table[c >> 1];
+    const float partner = to_float(src[c ^ 1]);
+    return (c & 1) == 0 ? v * cs.x - partner * cs.y : v * cs.x + partner * cs.y;
+  }
   const int half = dims >> 1;
   const bool low = c < half;
   const float2 cs = table[low ? c : c - half];
@@ -38,7 +43,7 @@ template <typename T>
 __global__ void latent_prepare_kernel(const T* __restrict__ proj, int ld, int q_col, int dkv_col, int heads, int dim, int rot,
                                       int rank, const int* __restrict__ slots, const void* __restrict__ norm_weight,
                                       int weight_dtype, float eps, const float2* __restrict__ cos_sin, int rot_dims,
-                                      T* __restrict__ cache, T* __restrict__ q_full, int n_tokens) {
+                                      T* __restrict__ cache, T* __restrict__ q_full, int n_tokens, int interleaved) {
   grid_dependency_wait();
   grid_dependency_launch();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -50,7 +55,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ proj, int ld, int q_
   if (which < heads) {
     const T* src = proj + (size_t)n * ld + q_col + (size_t)which * (dim + rot) + dim;
     T* dst = q_full + ((size_t)n * heads + which) * dk + rank;
-    for (int c = lane; c < rot; c += 32) dst[c] = from_float<T>(rotated(src, c, rot_dims, table));
+    for (int c = lane; c < rot; c += 32) dst[c] = from_float<T>(rotated(src, c, rot_dims, table, interleaved));
     return;
   }
   const int slot = slots[n];
@@ -66,7 +71,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ proj, int ld, int q_
   const float inv = 1.0f / sqrtf(sum_sq / (float)rank + eps);
   for (int c = lane; c < rank; c += 32)
     dst[c] = from_float<T>(load_as_float(norm_weight, weight_dtype, c) * (to_float(src[c]) * inv));
-  for (int c = lane; c < rot; c += 32) dst[rank + c] = from_float<T>(rotated(src + rank, c, rot_dims, table));
+  for (int c = lane; c < rot; c += 32) dst[rank + c] = from_float<T>(rotated(src + rank, c, rot_dims, table, interleaved));
 }
 
 __device__ __forceinline__ float latent_dot(const float* q_s, const float* row, int d) {
@@ -222,7 +227,7 @@ using namespace ms;
 MS_EXPORT int ms_latent_prepare(const void* proj, int dtype, int ld, int q_col, int dkv_col, int heads, int dim, int rot,
                                 int rank, const int* slots, const void* norm_weight, int weight_dtype, float eps,
                                 const float* cos_sin, int rot_dims, void* cache, void* q_full, int n_tokens,
-                                cudaStream_t stream) {
+                                int interleaved, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   MS_REQUIRE(heads > 0 && dim >= 0 && rot >= 0 && rank > 0, "latent_prepare: sizes must be positive (heads %d dim %d rot %d rank %d)",
              heads, dim, rot, rank);
@@ -235,7 +240,7 @@ MS_EXPORT int ms_latent_prepare(const void* proj, int dtype, int ld, int q_col, 
   MS_REQUIRE(blocks < 2147483647LL, "latent_prepare: %lld items in one launch is too many", items);
   MS_LAT_DISPATCH(dtype, (ms::launch(latent_prepare_kernel<T>, (unsigned)blocks, warps * 32, 0, stream, (const T*)proj, ld, q_col,
                                      dkv_col, heads, dim, rot, rank, slots, norm_weight, weight_dtype, eps,
-                                     (const float2*)cos_sin, rot_dims, (T*)cache, (T*)q_full, n_tokens)));
+                                     (const float2*)cos_sin, rot_dims, (T*)cache, (T*)q_full, n_tokens, interleaved)));
   MS_CHECK_LAUNCH("latent_prepare");
   return 0;
 }

@@ -1,6 +1,7 @@
 // Paged grouped-query attention on the tensor cores for head sizes that attention_mma.cu is not built for: query and key
 // heads of d entries and value heads of dv entries, both any multiple of 16 up to 128 and not necessarily the same, with
-// the two options of the other kernels (a sink in the softmax's denominator, a gate per head on the output).
+// the two options of the other kernels (a sink in the softmax's denominator, of score 0 or of a score per head; a gate per head
+// on the output).
 //
 // The scheme is attention_mma.cu's: one thread block per (request, key/value head, tile of query rows, split of the keys);
 // the rows of a tile are the pairs (token, query head of the kv head's group), token-major; W warps of 16 rows each; key and
@@ -22,6 +23,7 @@ attention_mma_any_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
                          const int* __restrict__ query_start, const int* __restrict__ context_lens, int page_size, int n_q,
                          int n_kv, int d, int dv, float scale_log2, int window, __nv_bfloat16* __restrict__ out,
                          float* __restrict__ part_o, float* __restrict__ part_lse, int num_splits, int sink,
+                         const float* __restrict__ sink_scores,
                          const __nv_bfloat16* __restrict__ gate, int gate_ld, int chunk, int n_v) {
   grid_dependency_wait();
   grid_dependency_launch();
@@ -73,7 +75,7 @@ attention_mma_any_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
         if (sink && split == 0) {                         // the sink alone: a result of zeros with weight 1
           float* dst = part_o + index * num_splits * dv;
           for (int c = 0; c < dv; ++c) dst[c] = 0.f;
-          part_lse[index * num_splits] = 0.f;
+          part_lse[index * num_splits] = sink_scores ? sink_scores[kv_head * group + row % group] * 1.4426950408889634f : 0.f;
         } else {
           part_lse[index * num_splits + split] = -INFINITY;
         }
@@ -234,8 +236,10 @@ attention_mma_any_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     const int row = thread_row(half);
     if (row >= rows_total) continue;
     const float m = m_run[half];
-    if (sink && split == 0) l += m == -INFINITY ? 1.f : exp2f(-m * scale_log2);
-    float inv = l > 0.f ? 1.f / l : 0.f;
+    float top = m == -INFINITY ? 0.f : m * scale_log2, kept = 1.f;
+    if (sink && split == 0)
+      kept = add_sink(m != -INFINITY, top, l, sink_scores ? sink_scores[kv_head * group + row % group] * 1.4426950408889634f : 0.f);
+    float inv = l > 0.f ? kept / l : 0.f;
     const size_t index = index_of(row);
     if (num_splits == 1) {
       if (gate != nullptr) inv /= 1.f + __expf(-__bfloat162float(gate[(size_t)(q0 + row / group) * gate_ld + kv_head * group + row % group]));
@@ -251,7 +255,7 @@ attention_mma_any_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
         if (n < dv / 8)
           *reinterpret_cast<float2*>(dst + n * 8 + quad_col * 2) = make_float2(acc_o[n][2 * half] * inv, acc_o[n][2 * half + 1] * inv);
       if (quad_col == 0)
-        part_lse[index * num_splits + split] = l > 0.f ? (m == -INFINITY ? 0.f : m * scale_log2) + log2f(l) : -INFINITY;
+        part_lse[index * num_splits + split] = l > 0.f ? top + log2f(l) : -INFINITY;
     }
   }
 }
@@ -284,7 +288,7 @@ template <int W, int BN>
 int launch_attention_any(const void* q, const void* k_pool, const void* v_pool, const int* block_tables, int table_stride,
                          const int* query_start, const int* context_lens, int page_size, int n_q, int n_kv, int d, int dv,
                          float scale, int window, void* out, float* part_o, float* part_lse, int num_splits, int n_requests,
-                         int max_query_len, int n_tokens, int sink, const void* gate, int gate_ld, int first_token,
+                         int max_query_len, int n_tokens, int sink, const float* sink_scores, const void* gate, int gate_ld, int first_token,
                          int chunk, int n_v, cudaStream_t stream) {
   constexpr int BM = 16 * W;
   const size_t smem = (size_t)(BM * (d + 8) + 2 * BN * (d + 8) + 2 * BN * (dv + 8)) * sizeof(__nv_bfloat16) + 4 * BN * sizeof(long long);
@@ -303,7 +307,7 @@ int launch_attention_any(const void* q, const void* k_pool, const void* v_pool, 
   dim3 grid((unsigned)tiles, n_kv, n_requests * num_splits);
   ms::launch(kernel, grid, W * 32, smem, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool,
              block_tables, table_stride, query_start, context_lens, page_size, n_q, n_kv, d, dv, scale * 1.4426950408889634f, window,
-             (__nv_bfloat16*)out, part_o, part_lse, num_splits, sink, (const __nv_bfloat16*)gate, gate_ld, chunk, n_v);
+             (__nv_bfloat16*)out, part_o, part_lse, num_splits, sink, sink_scores, (const __nv_bfloat16*)gate, gate_ld, chunk, n_v);
   MS_CHECK_LAUNCH("attention_mma_any");
   if (num_splits > 1) {
     const size_t skip = (size_t)first_token * n_q;
@@ -346,7 +350,8 @@ MS_EXPORT int ms_paged_attention_mma_any(const void* q, const void* k_pool, cons
                                          int table_stride, const int* query_start, const int* context_lens, int page_size,
                                          int n_q, int n_kv, int d, int dv, float scale, int window, void* out, float* part_o,
                                          float* part_lse, int num_splits, int n_requests, int max_query_len, int n_tokens,
-                                         int sink, const void* gate, int gate_ld, int first_token, int chunk, int n_v, cudaStream_t stream) {
+                                         int sink, const float* sink_scores, const void* gate, int gate_ld, int first_token, int chunk,
+                                         int n_v, cudaStream_t stream) {
   if (n_tokens == 0 || n_requests == 0) return 0;
   MS_REQUIRE(ms_attention_mma_any_supports(d, dv), "attention (any head size): sizes %d and %d are not multiples of 16 up to %d", d, dv, kAnyMax);
   MS_REQUIRE(n_kv > 0 && n_q % n_kv == 0, "attention: %d query heads are not a multiple of %d key/value heads", n_q, n_kv);
@@ -358,8 +363,8 @@ MS_EXPORT int ms_paged_attention_mma_any(const void* q, const void* k_pool, cons
   if (small)
     return launch_attention_any<1, 32>(q, k_pool, v_pool, block_tables, table_stride, query_start, context_lens, page_size, n_q, n_kv, d,
                                        dv, scale, window, out, part_o, part_lse, num_splits, n_requests, max_query_len, n_tokens, sink,
-                                       gate, gate_ld, first_token, chunk, n_v, stream);
+                                       sink_scores, gate, gate_ld, first_token, chunk, n_v, stream);
   return launch_attention_any<4, 64>(q, k_pool, v_pool, block_tables, table_stride, query_start, context_lens, page_size, n_q, n_kv, d, dv,
-                                     scale, window, out, part_o, part_lse, num_splits, n_requests, max_query_len, n_tokens, sink, gate,
+                                     scale, window, out, part_o, part_lse, num_splits, n_requests, max_query_len, n_tokens, sink, sink_scores, gate,
                                      gate_ld, first_token, chunk, n_v, stream);
 }

@@ -101,4 +101,15 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   return total;
 }
 
+// A sink in a row's softmax: one more term 2^sink2 of the denominator that has no value (sink2: its score times log2 e).  `top` is the
+// row's running maximum in base 2 (meaningless where nothing was seen: `seen` false) and `l` its sum relative to 2^top; both
+// become those of the row with the sink.  Returns the factor of what was accumulated relative to the old maximum.
+__device__ __forceinline__ float add_sink(bool seen, float& top, float& l, float sink2) {
+  const float new_top = seen ? fmaxf(top, sink2) : sink2;
+  const float factor = seen ? exp2f(top - new_top) : 0.f;
+  l = l * factor + exp2f(sink2 - new_top);
+  top = new_top;
+  return factor;
+}
+
 }  // namespace ms

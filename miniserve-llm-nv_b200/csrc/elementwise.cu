@@ -196,7 +196,7 @@ __global__ void qk_norm_rope_append_kernel(const T* __restrict__ qkv, const int*
 // ---------------------------------------------------------------- gated activation
 // out[n, c] = silu(gate_up[n, c]) * gate_up[n, inter + c]
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total) {
+__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total, float limit) {
   grid_dependency_wait();
   grid_dependency_launch();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -205,7 +205,7 @@ __global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ o
   const int c = (int)(i % inter);
   const float g = to_float(gate_up[n * 2 * inter + c]);
   const float u = to_float(gate_up[n * 2 * inter + inter + c]);
-  out[i] = from_float<T>(g / (1.0f + expf(-g)) * u);
+  out[i] = from_float<T>(limit > 0.f ? clamped_times(g, u, limit) : g / (1.0f + expf(-g)) * u);
 }
 
 }  // namespace ms
@@ -330,7 +330,9 @@ MS_EXPORT int ms_qk_norm_rope_append(const void* qkv, int dtype, const int* slot
 }
 
 // paired != 0: gate and up columns alternate in blocks of eight (inter must be a multiple of 8 then).
-MS_EXPORT int ms_silu_mul(const void* gate_up, int dtype, void* out, int n_tokens, int inter, int paired, cudaStream_t stream) {
+// limit > 0: the clamped gated activation in place of silu(gate) * up.
+MS_EXPORT int ms_silu_mul(const void* gate_up, int dtype, void* out, int n_tokens, int inter, int paired, float limit,
+                          cudaStream_t stream) {
   const size_t total = (size_t)n_tokens * inter;
   if (total == 0) return 0;
   MS_REQUIRE(!paired || inter % 8 == 0, "silu_mul: paired columns need a multiple of 8 features, not %d", inter);
@@ -339,14 +341,14 @@ MS_EXPORT int ms_silu_mul(const void* gate_up, int dtype, void* out, int n_token
     const size_t blocks8 = (total8 + 255) / 256;
     MS_REQUIRE(blocks8 < 2147483647ULL, "silu_mul: %zu elements in one launch is too many", total);
     MS_DISPATCH(dtype, (ms::launch(silu_mul_vec_kernel<T>, (unsigned)blocks8, 256, 0, stream, (const T*)gate_up, (T*)out, inter,
-                                                                                    total8, paired)));
+                                                                                    total8, paired, limit)));
     MS_CHECK_LAUNCH("silu_mul");
     return 0;
   }
   const size_t blocks = (total + 255) / 256;
   MS_REQUIRE(blocks < 2147483647ULL, "silu_mul: %zu elements in one launch is too many", total);
   MS_DISPATCH(dtype, (ms::launch(silu_mul_kernel<T>, (unsigned)blocks, 256, 0, stream, (const T*)gate_up, (T*)out, inter,
-                                                                             total)));
+                                                                             total, limit)));
   MS_CHECK_LAUNCH("silu_mul");
   return 0;
 }

@@ -7,6 +7,8 @@
 //   ms_qkv_prepare            per-head norm, partial half-split rotation and paged append for a projection whose columns are
 //                             laid out freely: query heads of d numbers, key heads of d, value heads of dv (another size),
 //                             or queries alone (a layer that reads another layer's keys and values)
+//   ms_qkv_prepare_rows       the same where queries and keys are normed over ALL their heads at once, with a temperature of the
+//                             queries that grows with the position
 //
 // All arithmetic is float32; storage is float32 or bfloat16.
 #include "common.cuh"
@@ -218,6 +220,109 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, int q_col
   }
 }
 
+// One block per token, for layers whose norm of queries and keys runs over the whole projection:
+//   q_out[n, h, c]  = t(p) * rotate(w_q[i] * q[n, i] / sqrt(mean(q[n]^2) + eps))    i = h d + c, the mean over all n_q d entries
+//   key pool        =        rotate(w_k[i] * k[n, i] / sqrt(mean(k[n]^2) + eps))    likewise over n_kv d entries
+//   value pool      =        v[n]
+// with t(p) = 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) at position p (temp_every <= 0: 1).  Columns, pools, slots and
+// rotation as qkv_prepare_kernel's; null weights: no norm.  `wide`: no rotation, head sizes and columns are multiples of eight
+// and every array lies on 16-byte boundaries: pieces of eight numbers.
+template <typename T>
+__global__ void qkv_prepare_rows_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col, int v_col, int n_q, int n_kv,
+                                        int d, int dv, const int* __restrict__ slots, const float* __restrict__ q_weight,
+                                        const float* __restrict__ k_weight, float eps, const float2* __restrict__ cos_sin,
+                                        int rotary_dim, int interleaved, const int* __restrict__ positions, float temp_coef,
+                                        double temp_every, T* __restrict__ k_pool, T* __restrict__ v_pool, int page_size,
+                                        T* __restrict__ q_out, int wide) {
+  grid_dependency_wait();
+  grid_dependency_launch();
+  __shared__ float scratch[32];
+  const size_t n = blockIdx.x;
+  const T* row = proj + n * ld;
+  const T *q = row + q_col, *k = row + k_col, *v = row + v_col;
+  const int q_size = n_q * d, k_size = n_kv * d, v_size = n_kv * dv;
+  float q_sq = 0.f, k_sq = 0.f;
+  if (wide) {
+    if (q_weight)
+      for (int i = threadIdx.x * 8; i < q_size; i += blockDim.x * 8) {
+        const Vec8 x = load8(q + i);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) q_sq += x.v[e] * x.v[e];
+      }
+    if (k_weight)
+      for (int i = threadIdx.x * 8; i < k_size; i += blockDim.x * 8) {
+        const Vec8 x = load8(k + i);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) k_sq += x.v[e] * x.v[e];
+      }
+  } else {
+    if (q_weight)
+      for (int i = threadIdx.x; i < q_size; i += blockDim.x) q_sq += to_float(q[i]) * to_float(q[i]);
+    if (k_weight)
+      for (int i = threadIdx.x; i < k_size; i += blockDim.x) k_sq += to_float(k[i]) * to_float(k[i]);
+  }
+  float q_factor = 1.f, k_factor = 1.f;
+  if (q_weight) q_factor = 1.0f / sqrtf(block_sum(q_sq, scratch) / (float)q_size + eps);
+  if (k_weight) k_factor = 1.0f / sqrtf(block_sum(k_sq, scratch) / (float)k_size + eps);
+  if (temp_every > 0.0) q_factor *= 1.f + temp_coef * logf((float)(floor((double)(positions[n] + 1) / temp_every) + 1.0));
+  const int slot = slots[n];
+  const int page = slot < 0 ? 0 : slot / page_size, offset = slot < 0 ? 0 : slot % page_size;
+  if (wide) {
+    for (int i = threadIdx.x * 8; i < q_size; i += blockDim.x * 8) {
+      Vec8 x = load8(q + i);
+      if (q_weight) {
+        const Vec8 w = load8(q_weight + i);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x.v[e] *= w.v[e];
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x.v[e] *= q_factor;
+      store8(q_out + n * q_size + i, x);
+    }
+    if (slot < 0) return;
+    for (int i = threadIdx.x * 8; i < k_size; i += blockDim.x * 8) {
+      Vec8 x = load8(k + i);
+      if (k_weight) {
+        const Vec8 w = load8(k_weight + i);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x.v[e] *= w.v[e] * k_factor;
+      }
+      const int g = i / d;
+      store8(k_pool + (((size_t)page * n_kv + g) * page_size + offset) * d + (i - g * d), x);
+    }
+    for (int i = threadIdx.x * 8; i < v_size; i += blockDim.x * 8) {
+      const int g = i / dv;
+      store8(v_pool + (((size_t)page * n_kv + g) * page_size + offset) * dv + (i - g * dv), load8(v + i));
+    }
+    return;
+  }
+  const int half = rotary_dim >> 1;
+  const float2* table = cos_sin ? cos_sin + n * half : nullptr;
+  auto value = [&](const T* src, const float* weight, float factor, int i) {      // entry i of a normed row, rotated
+    const int c = i % d;
+    float x = to_float(src[i]) * factor * (weight ? weight[i] : 1.f);
+    if (table && c < rotary_dim) {
+      const bool first = interleaved ? (c & 1) == 0 : c < half;
+      const int j = interleaved ? c >> 1 : (first ? c : c - half);
+      const int other_i = i - c + (interleaved ? c ^ 1 : (first ? c + half : c - half));
+      const float other = to_float(src[other_i]) * factor * (weight ? weight[other_i] : 1.f);
+      const float2 cs = table[j];
+      x = first ? x * cs.x - other * cs.y : x * cs.x + other * cs.y;
+    }
+    return x;
+  };
+  for (int i = threadIdx.x; i < q_size; i += blockDim.x) q_out[n * q_size + i] = from_float<T>(value(q, q_weight, q_factor, i));
+  if (slot < 0) return;
+  for (int i = threadIdx.x; i < k_size; i += blockDim.x) {
+    const int g = i / d;
+    k_pool[(((size_t)page * n_kv + g) * page_size + offset) * d + (i - g * d)] = from_float<T>(value(k, k_weight, k_factor, i));
+  }
+  for (int i = threadIdx.x; i < v_size; i += blockDim.x) {
+    const int g = i / dv;
+    v_pool[(((size_t)page * n_kv + g) * page_size + offset) * dv + (i - g * dv)] = v[i];
+  }
+}
+
 }  // namespace ms
 
 using namespace ms;
@@ -281,6 +386,29 @@ MS_EXPORT int ms_qkv_prepare(const void* proj, int dtype, int ld, int q_col, int
                                     k_col, v_col, n_q, n_kv, d, dv, slots, q_weight, k_weight, eps, (const float2*)cos_sin,
                                     rotary_dim, (T*)k_pool, (T*)v_pool, page_size, (T*)q_out, n_tokens, interleaved, bias, value_heads > 0 ? value_heads : n_kv)));
   MS_CHECK_LAUNCH("qkv_prepare");
+  return 0;
+}
+
+// proj [n_tokens, ld]; norm weights float32 [n_q d] and [n_kv d] (null: no norm); positions int32 [n_tokens] (read where temp_every > 0).
+MS_EXPORT int ms_qkv_prepare_rows(const void* proj, int dtype, int ld, int q_col, int k_col, int v_col, int n_q, int n_kv, int d,
+                                  int dv, const int* slots, const float* q_weight, const float* k_weight, float eps,
+                                  const float* cos_sin, int rotary_dim, int interleaved, const int* positions, float temp_coef,
+                                  float temp_every, void* k_pool, void* v_pool, int page_size, void* q_out, int n_tokens,
+                                  cudaStream_t stream) {
+  if (n_tokens == 0) return 0;
+  MS_REQUIRE(d > 0 && dv > 0 && n_q > 0 && n_kv > 0 && page_size > 0, "qkv_prepare_rows: %d/%d heads of %d/%d, pages of %d", n_q, n_kv, d, dv, page_size);
+  MS_REQUIRE(rotary_dim >= 0 && rotary_dim <= d && rotary_dim % 2 == 0 && (rotary_dim == 0 || cos_sin),
+             "qkv_prepare_rows: rotary size %d must be even, at most the head size %d and have its table", rotary_dim, d);
+  MS_REQUIRE(temp_every <= 0.f || positions, "qkv_prepare_rows: a temperature by position needs the positions");
+  auto aligned = [](const void* p) { return reinterpret_cast<size_t>(p) % 16 == 0; };
+  const int wide = rotary_dim == 0 && d % 8 == 0 && dv % 8 == 0 && ld % 8 == 0 && q_col % 8 == 0 && k_col % 8 == 0 && v_col % 8 == 0 &&
+                   aligned(proj) && aligned(q_out) && aligned(k_pool) && aligned(v_pool) && aligned(q_weight) && aligned(k_weight);
+  const int threads = n_q * d >= 2048 ? 256 : 128;
+  MS_EG_DISPATCH(dtype, (ms::launch(qkv_prepare_rows_kernel<T>, n_tokens, threads, 0, stream, (const T*)proj, ld, q_col, k_col, v_col,
+                                    n_q, n_kv, d, dv, slots, q_weight, k_weight, eps, (const float2*)(rotary_dim ? cos_sin : nullptr),
+                                    rotary_dim, interleaved, positions, temp_coef, (double)temp_every, (T*)k_pool, (T*)v_pool,
+                                    page_size, (T*)q_out, wide)));
+  MS_CHECK_LAUNCH("qkv_prepare_rows");
   return 0;
 }
 
@@ -384,6 +512,22 @@ __global__ void sigmoid_gate_mul_kernel(const T* __restrict__ x, const T* __rest
   out[i] = from_float<T>(to_float(x[i]) / (1.f + expf(-g)));
 }
 
+// The same in pieces of eight numbers, where the width, the gate's place and its rows are multiples of eight on 16-byte boundaries.
+template <typename T>
+__global__ void sigmoid_gate_mul_vec_kernel(const T* __restrict__ x, const T* __restrict__ gate, int gate_ld, int gate_col,
+                                            T* __restrict__ out, size_t pieces, int per_row) {
+  grid_dependency_wait();
+  grid_dependency_launch();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= pieces) return;
+  const size_t n = i / per_row;
+  const Vec8 g = load8(gate + n * gate_ld + gate_col + (i - n * per_row) * 8);
+  Vec8 v = load8(x + i * 8);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v.v[e] /= 1.f + expf(-g.v[e]);
+  store8(out + i * 8, v);
+}
+
 // One warp per (token, head): o = first - lambda second with first = a[n, head], second = a[n, heads + head] (the outputs of
 // two score maps over the same values), o / sqrt(mean(o^2) + eps) * out_scale * sigmoid(gate[n, gate_col + head dv + c]).
 // `wide`: dv is a multiple of four, at most 512, and every row lies on a boundary of four numbers: a lane keeps its pieces of
@@ -470,6 +614,15 @@ MS_EXPORT int ms_sigmoid_gate_mul(const void* x, const void* gate, int gate_ld, 
                                   int width, cudaStream_t stream) {
   const long long total = (long long)rows * width;
   if (total == 0) return 0;
+  if (width % 8 == 0 && gate_ld % 8 == 0 && gate_col % 8 == 0 && reinterpret_cast<size_t>(x) % 16 == 0 &&
+      reinterpret_cast<size_t>(gate) % 16 == 0 && reinterpret_cast<size_t>(out) % 16 == 0) {
+    const long long pieces = total / 8, piece_blocks = (pieces + 127) / 128;
+    MS_REQUIRE(piece_blocks < 2147483647LL, "sigmoid_gate_mul: %lld elements in one launch is too many", total);
+    MS_EG_DISPATCH(dtype, (ms::launch(sigmoid_gate_mul_vec_kernel<T>, (unsigned)piece_blocks, 128, 0, stream, (const T*)x, (const T*)gate,
+                                      gate_ld, gate_col, (T*)out, (size_t)pieces, width / 8)));
+    MS_CHECK_LAUNCH("sigmoid_gate_mul");
+    return 0;
+  }
   const long long blocks = (total + 255) / 256;
   MS_REQUIRE(blocks < 2147483647LL, "sigmoid_gate_mul: %lld elements in one launch is too many", total);
   MS_EG_DISPATCH(dtype, (ms::launch(sigmoid_gate_mul_kernel<T>, (unsigned)blocks, 256, 0, stream, (const T*)x, (const T*)gate, gate_ld,

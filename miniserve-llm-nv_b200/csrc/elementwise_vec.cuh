@@ -308,8 +308,15 @@ __device__ __forceinline__ float silu_times(float g, float u) {
   return g / (1.0f + expf(-g)) * u;
 }
 
+// The clamped gated activation: g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = clamp(up, -limit, limit).
+__device__ __forceinline__ float clamped_times(float gate, float up, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
 template <typename T>
-__global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total8, int paired) {
+__global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total8, int paired,
+                                    float limit) {
   grid_dependency_wait();
   grid_dependency_launch();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -329,7 +336,7 @@ __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict
   const Vec8 u = load8(row + (paired ? 2 * c + 8 : inter + c));
   Vec8 y;
 #pragma unroll
-  for (int e = 0; e < 8; ++e) y.v[e] = silu_times<T>(g.v[e], u.v[e]);
+  for (int e = 0; e < 8; ++e) y.v[e] = limit > 0.f ? clamped_times(g.v[e], u.v[e], limit) : silu_times<T>(g.v[e], u.v[e]);
   store8(out + n * inter + c, y);
 }
 

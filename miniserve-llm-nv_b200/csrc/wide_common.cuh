@@ -41,6 +41,19 @@ __device__ __forceinline__ float silu_times(float g, float u) {
   return g * (g >= 0.f ? r : e * r) * u;
 }
 
+// The clamped gated activation, g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = clamp(up, -limit, limit).
+__device__ __forceinline__ float clamped_times(float gate, float up, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  const float e = __expf(-1.702f * fabsf(g));
+  const float r = __fdividef(1.0f, 1.0f + e);
+  return g * (g >= 0.f ? r : e * r) * (u + 1.f);
+}
+
+// A gated activation: silu(g) u, or the clamped one where a limit (above 0) is given.
+__device__ __forceinline__ float gated_times(float g, float u, float limit) {
+  return limit > 0.f ? clamped_times(g, u, limit) : silu_times(g, u);
+}
+
 // Barriers of the computing warps alone (the copying warp takes no part).
 __device__ __forceinline__ bool all_compute_warps(bool ok) {
   unsigned all;

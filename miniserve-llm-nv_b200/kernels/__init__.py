@@ -10,13 +10,13 @@ from __future__ import annotations
 
 import ctypes
 import logging
-from typing import Optional
+from typing import Optional, Union
 
 import torch
 
 from . import build
 
-ABI_VERSION = 11
+ABI_VERSION = 12
 log = logging.getLogger("miniserve_b200")
 _library: Optional[ctypes.CDLL] = None
 
@@ -182,6 +182,55 @@ def postnorm_add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], 
         _i(_code(weight.dtype)) if weight is not None else 0, _f(eps), _ptr(rows), _ptr(out), _i(n_out), _i(hidden), _stream()))
 
 
+def add_layernorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, bias: torch.Tensor, eps: float,
+                  out: torch.Tensor, rows: Optional[torch.Tensor] = None, delta2: Optional[torch.Tensor] = None,
+                  vector: Optional[torch.Tensor] = None, weight2: Optional[torch.Tensor] = None,
+                  bias2: Optional[torch.Tensor] = None, out2: Optional[torch.Tensor] = None) -> None:
+    """Adds ``delta`` (or ``delta + delta2``, summed in float32) and ``vector`` (float32 ``[H]``, the same for every row) into the
+    float32 ``residual`` (in place) and writes its layer norm to ``out``: ``weight * (x - mean) / sqrt(mean((x - mean)^2) + eps) +
+    bias``.  With ``out2`` the same normed row is written a second time with ``weight2`` and ``bias2``.  With ``rows`` (int32
+    ``[K]``) only those rows are normed, into ``out [K, H]``, and the residual is left untouched.  The weights and biases share
+    one type, float32 or bfloat16, whatever ``out`` is."""
+    hidden = residual.shape[1]
+    n_out = residual.shape[0] if rows is None else rows.numel()
+    _want(residual, "residual", torch.float32)
+    _want(out, "out", None, (n_out, hidden))
+    _want(weight, "weight", None, (hidden,))
+    _want(bias, "bias", weight.dtype, (hidden,))
+    if delta is None and delta2 is not None:
+        delta, delta2 = delta2, None
+    for name, tensor in (("delta", delta), ("delta2", delta2)):
+        if tensor is not None:
+            _want(tensor, name, out.dtype, residual.shape)
+    if vector is not None:
+        _want(vector, "vector", torch.float32, (hidden,))
+    if out2 is not None:
+        _want(out2, "out2", out.dtype, (n_out, hidden))
+        _want(weight2, "weight2", weight.dtype, (hidden,))
+        _want(bias2, "bias2", weight.dtype, (hidden,))
+    if rows is not None:
+        _want(rows, "rows", torch.int32)
+    _check(library().ms_add_layernorm(
+        _ptr(residual), _ptr(delta), _ptr(delta2), _i(_code(out.dtype)), _ptr(vector), _ptr(weight), _ptr(bias), _ptr(weight2),
+        _ptr(bias2), _i(_code(weight.dtype)), _f(eps), _ptr(rows), _ptr(out), _ptr(out2), _i(n_out), _i(hidden), _stream()))
+
+
+def stream_to_columns(residual: torch.Tensor, delta: Optional[torch.Tensor], out: torch.Tensor, col: int,
+                      delta2: Optional[torch.Tensor] = None) -> None:
+    """``out[n, col : col + H] = residual[n] + (delta[n] + delta2[n])`` rounded once to ``out``'s type: the stream with what is
+    still to be added, as columns of a wider matrix ``out [N, ld]``.  The residual is left as it is."""
+    n, hidden = residual.shape
+    _want(residual, "residual", torch.float32)
+    _want(out, "out")
+    if out.dim() != 2 or out.shape[0] != n or col < 0 or col + hidden > out.shape[1]:
+        raise KernelError(f"stream_to_columns: columns {col} .. {col + hidden} of {tuple(out.shape)} for {n} rows")
+    for name, tensor in (("delta", delta), ("delta2", delta2)):
+        if tensor is not None:
+            _want(tensor, name, out.dtype, residual.shape)
+    _check(library().ms_stream_to_columns(_ptr(residual), _ptr(delta), _ptr(delta2), _i(_code(out.dtype)), _ptr(out), _i(out.shape[1]),
+                                          _i(col), _i(n), _i(hidden), _stream()))
+
+
 def qkv_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, n_q: int, n_kv: int, head_dim: int, value_dim: int,
                 slots: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
                 cos_sin: Optional[torch.Tensor], rotary_dim: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
@@ -230,6 +279,45 @@ def qkv_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, n_q: int
         _i(k_pool.shape[2]) if own else 1, _ptr(q_out), _i(n), _i(1 if interleaved else 0), _ptr(bias), _i(value_heads), _stream()))
 
 
+def qkv_prepare_rows(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, n_q: int, n_kv: int, head_dim: int, value_dim: int,
+                     slots: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
+                     cos_sin: Optional[torch.Tensor], rotary_dim: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
+                     q_out: torch.Tensor, interleaved: bool = False, positions: Optional[torch.Tensor] = None,
+                     temperature: Optional[tuple] = None) -> None:
+    """:func:`qkv_prepare` for layers whose RMSNorm of queries and of keys runs over all heads at once: the weights are float32
+    ``[n_q * head_dim]`` and ``[n_kv * head_dim]`` (None: no norm), the mean square is taken over the whole row.
+    ``temperature`` (coef, every): the queries of a token at position p are multiplied by ``1 + coef * ln(floor((p + 1) / every) +
+    1)``, after norm and rotation, in float32; it needs ``positions`` (int32 ``[N]``)."""
+    n, ld = proj.shape
+    _want(proj, "proj")
+    _want(q_out, "q_out", proj.dtype, (n, n_q, head_dim))
+    if (min(q_col, k_col, v_col) < 0 or q_col + n_q * head_dim > ld or k_col + n_kv * head_dim > ld or v_col + n_kv * value_dim > ld):
+        raise KernelError(f"qkv_prepare_rows: columns {q_col}, {k_col}, {v_col} of {n_q}/{n_kv} heads of {head_dim}/{value_dim} in rows of {ld}")
+    _want(slots, "slots", torch.int32, (n,))
+    _want(k_pool, "k_pool", proj.dtype)
+    _want(v_pool, "v_pool", proj.dtype)
+    if (k_pool.dim() != 4 or tuple(k_pool.shape[1:]) != (n_kv, k_pool.shape[2], head_dim)
+            or tuple(v_pool.shape) != (k_pool.shape[0], n_kv, k_pool.shape[2], value_dim)):
+        raise KernelError(f"pool shapes {tuple(k_pool.shape)}, {tuple(v_pool.shape)} are not [pages, {n_kv}, page_size, {head_dim} | {value_dim}]")
+    for name, weight, heads in (("q_weight", q_weight, n_q), ("k_weight", k_weight, n_kv)):
+        if weight is not None:
+            _want(weight, name, torch.float32, (heads * head_dim,))
+    if cos_sin is not None:
+        _want(cos_sin, "cos_sin", torch.float32, (n, rotary_dim // 2, 2))
+    else:
+        rotary_dim = 0
+    coef, every = (0.0, 0.0) if temperature is None else temperature
+    if temperature is not None:
+        if positions is None or every <= 0:
+            raise KernelError(f"qkv_prepare_rows: a temperature {temperature} needs the positions and a step above 0")
+        _want(positions, "positions", torch.int32, (n,))
+    _check(library().ms_qkv_prepare_rows(
+        _ptr(proj), _i(_code(proj.dtype)), _i(ld), _i(q_col), _i(k_col), _i(v_col), _i(n_q), _i(n_kv), _i(head_dim), _i(value_dim),
+        _ptr(slots), _ptr(q_weight), _ptr(k_weight), _f(eps), _ptr(cos_sin), _i(rotary_dim), _i(1 if interleaved else 0),
+        _ptr(positions) if temperature is not None else None, _f(coef), _f(every), _ptr(k_pool), _ptr(v_pool), _i(k_pool.shape[2]),
+        _ptr(q_out), _i(n), _stream()))
+
+
 def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, cos_sin: torch.Tensor, magnitude: float = 1.0) -> None:
     """``cos_sin[n, j] = magnitude * (cos, sin)(positions[n] * inv_freq[j])`` in float32; cos_sin ``[N, half, 2]``."""
     n, half = positions.numel(), inv_freq.numel()
@@ -274,9 +362,11 @@ def qk_norm_rope_append(qkv: torch.Tensor, slots: torch.Tensor, q_weight: Option
         _i(n_q), _i(n_kv), _i(head_dim), _ptr(q_out), _i(n), _stream()))
 
 
-def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, paired: bool = False, bias: Optional[torch.Tensor] = None) -> None:
+def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, paired: bool = False, bias: Optional[torch.Tensor] = None,
+             limit: Optional[float] = None) -> None:
     """``out[n, c] = silu(gate_up[n, c]) * gate_up[n, I + c]`` for gate_up ``[N, 2 I]``.  With ``bias`` (float32 ``[2 I]``,
-    not with ``paired``) it is added to both halves first, in float32.
+    not with ``paired``) it is added to both halves first, in float32.  ``limit`` (not with ``bias``): the clamped gated
+    activation instead, ``g sigmoid(1.702 g) (u + 1)`` with ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``.
 
     ``paired``: the columns come as :func:`interleave_gate_up` orders a weight's rows (eight gate columns, then
     the up columns of the same features, and so on): ``out[n, 8 j + r] = silu(gate_up[n, 16 j + r]) *
@@ -287,12 +377,12 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, paired: bool = False, bia
     _want(out, "out", gate_up.dtype)
     if bias is not None:
         _want(bias, "bias", torch.float32, (2 * inter,))
-        if paired:
-            raise KernelError("silu_mul: a bias goes with the plain layout (gate columns, then up columns)")
+        if paired or limit:
+            raise KernelError("silu_mul: a bias goes with the plain layout (gate columns, then up columns) and the plain activation")
         _check(library().ms_silu_mul_bias(_ptr(gate_up), _i(_code(gate_up.dtype)), _ptr(bias), _ptr(out), _i(n), _i(inter), _stream()))
         return
     _check(library().ms_silu_mul(_ptr(gate_up), _i(_code(gate_up.dtype)), _ptr(out), _i(n), _i(inter),
-                                 _i(1 if paired else 0), _stream()))
+                                 _i(1 if paired else 0), _f(limit or 0.0), _stream()))
 
 
 def add_bias(x: torch.Tensor, bias: torch.Tensor) -> None:
@@ -434,7 +524,8 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                     request_of_token: torch.Tensor, positions: torch.Tensor, query_start: torch.Tensor,
                     context_lens: torch.Tensor, max_query_len: int, max_context_len: int, scale: float,
                     window: Optional[int], out: torch.Tensor, host_query_start: Optional[list] = None,
-                    softcap: Optional[float] = None, bias_slopes: Optional[torch.Tensor] = None, sink: bool = False,
+                    softcap: Optional[float] = None, bias_slopes: Optional[torch.Tensor] = None,
+                    sink: Union[bool, torch.Tensor] = False,
                     gate: Optional[torch.Tensor] = None, gate_col: int = 0, chunk: Optional[int] = None) -> None:
     """Causal grouped-query attention of every token over its request's paged keys and values.
 
@@ -443,8 +534,8 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     ``g % value heads``.  The general kernel and the tensor-core kernel for any head size implement both.
 
     q ``[N, n_q, d]``, out ``[N, n_q, dv]`` (dv: the value pool's last dimension, usually d); pools of one layer
-    ``[pages, n_kv, page_size, d | dv]``.  ``sink``: the softmax's denominator gets one more term ``exp(0)`` (a key of
-    score 0 without a value).  ``gate [N, ld]`` with ``gate_col``: head h's output is multiplied by
+    ``[pages, n_kv, page_size, d | dv]``.  ``sink``: the softmax's denominator gets one more term, ``exp(0)`` (True: a key of
+    score 0 without a value) or ``exp(sink[h])`` (a float32 tensor ``[n_q]``: a score per query head, not scaled).  ``gate [N, ld]`` with ``gate_col``: head h's output is multiplied by
     ``sigmoid(gate[n, gate_col + h])`` as it is stored.  block_tables
     int32 ``[R, width]``; request_of_token, positions int32 ``[N]``; query_start ``[R + 1]`` and
     context_lens ``[R]`` describe the same batch per request (a request's tokens are the last
@@ -488,6 +579,10 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     _want(context_lens, "context_lens", torch.int32, (n_requests,))
     lib = library()
     n_kv = k_pool.shape[1]
+    sink_scores = None
+    if isinstance(sink, torch.Tensor):
+        _want(sink, "sink", torch.float32, (n_q,))
+        sink, sink_scores = True, sink
     modified = bool(softcap) or bias_slopes is not None
     if bias_slopes is not None:
         _want(bias_slopes, "bias_slopes", torch.float32, (n_q,))
@@ -498,7 +593,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     if (USE_MMA_ANY and extended and not modified and q.dtype == torch.bfloat16
             and (value_dim != head_dim or bool(chunk) or shared_values or not lib.ms_attention_mma_supports(_i(head_dim)))
             and lib.ms_attention_mma_any_supports(_i(head_dim), _i(value_dim))):
-        reach = min(max_context_len, chunk) if chunk else max_context_len      # the most keys a token sees
+        reach = min([max_context_len] + [limit for limit in (chunk, window) if limit])      # the most keys a token sees
         def run_any(first: int, last: int, longest: int, rows: int, first_row: int = 0) -> None:
             count = last - first
             splits = lib.ms_attention_mma_any_splits(_i(count), _i(n_kv), _i(n_q), _i(longest), _i(reach))
@@ -510,7 +605,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                 _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_tables[first:last]), _i(block_tables.shape[1]),
                 _ptr(query_start[first:last + 1]), _ptr(context_lens[first:last]), _i(k_pool.shape[2]), _i(n_q), _i(n_kv),
                 _i(head_dim), _i(value_dim), _f(scale), _i(window if window else 0), _ptr(out), _ptr(part_o), _ptr(part_lse),
-                _i(splits), _i(count), _i(longest), _i(rows), _i(1 if sink else 0), gate_ptr, _i(gate_ld), _i(first_row),
+                _i(splits), _i(count), _i(longest), _i(rows), _i(1 if sink else 0), _ptr(sink_scores), gate_ptr, _i(gate_ld), _i(first_row),
                 _i(chunk or 0), _i(n_v), _stream()))
 
         single = 0
@@ -529,7 +624,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
             _ptr(q), _i(_code(q.dtype)), _ptr(k_pool), _ptr(v_pool), _ptr(block_tables), _i(block_tables.shape[1]),
             _ptr(request_of_token), _ptr(positions), _i(k_pool.shape[2]), _i(n_q), _i(n_kv), _i(head_dim),
             _f(scale), _i(window if window else 0), _f(softcap if softcap else 0.0), _ptr(bias_slopes), _ptr(out),
-            _i(n), _i(value_dim), _i(1 if sink else 0), gate_ptr, _i(gate_ld), _i(chunk or 0), _i(n_v), _stream()))
+            _i(n), _i(value_dim), _i(1 if sink else 0), _ptr(sink_scores), gate_ptr, _i(gate_ld), _i(chunk or 0), _i(n_v), _stream()))
         return
 
     def run(first: int, last: int, longest: int, rows: int, first_row: int = 0) -> None:
@@ -549,7 +644,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                     _ptr(q), _ptr(k_pool), _ptr(v_pool), _i(k_pool.shape[0]), _ptr(tables), _i(block_tables.shape[1]),
                     _ptr(starts), _ptr(lens), _i(k_pool.shape[2]), _i(n_q), _i(n_kv), _i(head_dim), _f(scale),
                     _i(window if window else 0), _ptr(out), _i(count), _i(longest), _i(n),
-                    _ptr(device_error_flag(q.device)), _i(1 if sink else 0), gate_ptr, _i(gate_ld), _stream()))
+                    _ptr(device_error_flag(q.device)), _i(1 if sink else 0), _ptr(sink_scores), gate_ptr, _i(gate_ld), _stream()))
                 return
             _check(lib.ms_paged_attention_tcgen05(
                 _ptr(q), _ptr(k_pool), _ptr(v_pool), _i(k_pool.shape[0]), _ptr(tables), _i(block_tables.shape[1]),
@@ -565,8 +660,8 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
         _check(lib.ms_paged_attention_mma(
             _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(tables), _i(block_tables.shape[1]), _ptr(starts), _ptr(lens),
             _i(k_pool.shape[2]), _i(n_q), _i(n_kv), _i(head_dim), _f(scale), _i(window if window else 0), _ptr(out),
-            _ptr(part_o), _ptr(part_lse), _i(splits), _i(count), _i(longest), _i(rows), _i(1 if sink else 0), gate_ptr,
-            _i(gate_ld), _i(first_row), _stream()))
+            _ptr(part_o), _ptr(part_lse), _i(splits), _i(count), _i(longest), _i(rows), _i(1 if sink else 0), _ptr(sink_scores),
+            gate_ptr, _i(gate_ld), _i(first_row), _stream()))
 
     leading_single = 0
     if host_query_start and max_query_len > 1 and len(host_query_start) == n_requests + 1:
@@ -652,13 +747,14 @@ def decode_attention_fused(qkv: torch.Tensor, slots: torch.Tensor, q_weight: Opt
 
 def latent_prepare(proj: torch.Tensor, q_col: int, dkv_col: int, heads: int, dim: int, rot: int, rank: int,
                    slots: torch.Tensor, norm_weight: torch.Tensor, eps: float, cos_sin: Optional[torch.Tensor],
-                   rot_dims: int, cache: torch.Tensor, q_full: torch.Tensor) -> None:
+                   rot_dims: int, cache: torch.Tensor, q_full: torch.Tensor, interleaved: bool = False) -> None:
     """What a latent-attention layer does between its input projection and its attention, for every token:
     the latent ``proj[n, dkv_col : dkv_col + rank]`` is RMS-normed with ``norm_weight`` and, followed by the rotated
     key part ``proj[n, dkv_col + rank : + rot]``, written to row ``slots[n]`` of ``cache [pages, page_size, rank + rot]``
     (negative slot: no write); the rotated part of every query head (``proj[n, q_col + h (dim + rot) + dim : + rot]``)
     is rotated into ``q_full[n, h, rank:]``.  The rotation acts on the first ``rot_dims`` entries of a rotated part,
-    entry i paired with i + rot_dims / 2, by ``cos_sin`` float32 ``[N, rot_dims / 2, 2]``."""
+    entry i paired with i + rot_dims / 2 (``interleaved``: entry 2i with entry 2i + 1), by ``cos_sin`` float32
+    ``[N, rot_dims / 2, 2]``."""
     n, ld = proj.shape
     _want(proj, "proj")
     _want(slots, "slots", torch.int32, (n,))
@@ -675,7 +771,7 @@ def latent_prepare(proj: torch.Tensor, q_col: int, dkv_col: int, heads: int, dim
         rot_dims = 0
     _check(library().ms_latent_prepare(_ptr(proj), _i(_code(proj.dtype)), _i(ld), _i(q_col), _i(dkv_col), _i(heads), _i(dim),
                                        _i(rot), _i(rank), _ptr(slots), _ptr(norm_weight), _i(_code(norm_weight.dtype)), _f(eps),
-                                       _ptr(cos_sin), _i(rot_dims), _ptr(cache), _ptr(q_full), _i(n), _stream()))
+                                       _ptr(cos_sin), _i(rot_dims), _ptr(cache), _ptr(q_full), _i(n), _i(1 if interleaved else 0), _stream()))
 
 
 def latent_attention_kernels(dtype: torch.dtype, rank: int, rot: int, heads: int, page_size: int) -> dict:
@@ -713,8 +809,8 @@ def latent_attention(q_full: torch.Tensor, cache: torch.Tensor, block_tables: to
     lib = library()
     page_size = cache.shape[1]
     if q_full.dtype == torch.bfloat16 and USE_LATENT_MMA and lib.ms_latent_attention_mma_supports(_i(rank), _i(dk - rank), _i(heads)):
-        splits = lib.ms_latent_attention_mma_splits(_i(rank), _i(dk - rank), _i(heads), _i(n_requests), _i(max_query_len),
-                                                    _i(max_context_len))
+        reach = min(max_context_len, window) if window else max_context_len      # the most keys a token sees
+        splits = lib.ms_latent_attention_mma_splits(_i(rank), _i(dk - rank), _i(heads), _i(n_requests), _i(max_query_len), _i(reach))
         part_o = part_lse = None
         if splits > 1:
             part_o = torch.empty((n * heads * splits, rank), dtype=torch.float32, device=q_full.device)
@@ -1436,10 +1532,11 @@ PAIR_WIDE = __import__("os").environ.get("MINISERVE_B200_PAIR_WIDE", "0") == "1"
 
 
 def linear_pair(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, add: bool = False, gated: bool = False,
-                row_stats: Optional["RowStats"] = None, wide: Optional[bool] = None) -> None:
+                row_stats: Optional["RowStats"] = None, wide: Optional[bool] = None, limit: Optional[float] = None) -> None:
     """``out = x @ weight^T`` by the kernel in which two thread blocks share each 256 x 256 tile (tcgen05 with
     ``cta_group::2``).  ``add``: ``out += ...`` on a float32 ``out``.  ``gated``: ``weight`` is
-    :func:`interleave_gate_up` of a gate and an up projection and ``out [M, N / 2] = silu(gate) * up``.
+    :func:`interleave_gate_up` of a gate and an up projection and ``out [M, N / 2] = silu(gate) * up`` (``limit``: the
+    clamped activation of :func:`silu_mul`).
     ``row_stats`` (from :func:`linear_pair_residual`): ``x`` still lacks the division by its rows' root mean square,
     and the results are multiplied by it before they are rounded.
 
@@ -1463,7 +1560,7 @@ def linear_pair(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, add: b
                                   _i(1 if (PAIR_WIDE if wide is None else wide) else 0),
                                   _i(m), _i(n), _i(k), _ptr(row_stats.partials if row_stats else None),
                                   _i(row_stats.count if row_stats else 0), _f(row_stats.eps if row_stats else 0.0), None, None,
-                                  _i(0), None, _ptr(device_error_flag(x.device)), _stream()))
+                                  _i(0), None, _f(limit or 0.0), _ptr(device_error_flag(x.device)), _stream()))
 
 
 QKV_IN_PRODUCT = __import__("os").environ.get("MINISERVE_B200_QKV_IN_PRODUCT", "1") == "1"
@@ -1542,7 +1639,7 @@ def linear_pair_residual(x: torch.Tensor, weight: torch.Tensor, residual: torch.
         raise KernelError(f"linear_pair_residual: weight {tuple(weight.shape)}, partials {tuple(partials.shape)} for {tiles} "
                           f"tiles of {m} rows")
     _check(library().ms_gemm_pair(_ptr(x), _ptr(weight), _ptr(x_next), _i(1), _i(3), _i(0), _i(m), _i(n), _i(k), None, _i(0),
-                                  _f(0.0), _ptr(residual), _ptr(norm_weight), _i(_code(norm_weight.dtype)), _ptr(partials),
+                                  _f(0.0), _ptr(residual), _ptr(norm_weight), _i(_code(norm_weight.dtype)), _ptr(partials), _f(0.0),
                                   _ptr(device_error_flag(x.device)), _stream()))
     return RowStats(partials, tiles, eps, per_row=True)
 
@@ -1784,7 +1881,7 @@ def wide_blocks(n: int, k: int) -> int:
 
 
 def _wide_call(x, weight, out, out_code: int, mode: int, m: int, n: int, k: int, row_stats: Optional[RowStats],
-               residual=None, norm_weight=None, x_next=None, out_partials=None) -> None:
+               residual=None, norm_weight=None, x_next=None, out_partials=None, limit: Optional[float] = None) -> None:
     if row_stats is not None:
         _want(row_stats.partials, "row_stats.partials", torch.float32)
         if row_stats.partials.dim() != 2 or row_stats.partials.shape[1] != 8 or row_stats.partials.shape[0] < row_stats.count:
@@ -1793,18 +1890,18 @@ def _wide_call(x, weight, out, out_code: int, mode: int, m: int, n: int, k: int,
         _ptr(x), _ptr(weight), _ptr(out), _i(out_code), _i(mode), _i(m), _i(n), _i(k),
         _ptr(row_stats.partials if row_stats else None), _i(row_stats.count if row_stats else 0),
         _f(row_stats.eps if row_stats else 0.0), _ptr(residual), _ptr(norm_weight),
-        _i(_code(norm_weight.dtype) if norm_weight is not None else 0), _ptr(x_next), _ptr(out_partials),
+        _i(_code(norm_weight.dtype) if norm_weight is not None else 0), _ptr(x_next), _ptr(out_partials), _f(limit or 0.0),
         _ptr(device_error_flag(x.device)), _stream()))
 
 
 def linear_wide(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: bool = False,
-                row_stats: Optional[RowStats] = None) -> None:
+                row_stats: Optional[RowStats] = None, limit: Optional[float] = None) -> None:
     """``out = x @ weight^T`` for up to 8 rows of bfloat16 ``x`` by the library's kernel for weights of many
     rows (no sum across blocks); ``out`` bfloat16 or float32.
 
     ``gated``: ``weight [2 I, K]`` holds a gated feed-forward's two projections in blocks of sixteen rows,
     eight gate rows followed by the up rows of the same features (:func:`interleave_gate_up`), and
-    ``out [M, I]`` bfloat16 receives ``silu(gate) * up``.  ``row_stats``: ``x`` comes from
+    ``out [M, I]`` bfloat16 receives ``silu(gate) * up`` (``limit``: the clamped activation of :func:`silu_mul`).  ``row_stats``: ``x`` comes from
     :func:`linear_wide_residual`; its rows' norm is completed on the results (before the activation).
     """
     m, k = x.shape
@@ -1812,7 +1909,7 @@ def linear_wide(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated:
     _want(x, "x", torch.bfloat16)
     _want(weight, "weight", torch.bfloat16, (n, k))
     _want(out, "out", torch.bfloat16 if gated else None, (m, n // 2 if gated else n))
-    _wide_call(x, weight, out, _code(out.dtype), 1 if gated else 0, m, n, k, row_stats)
+    _wide_call(x, weight, out, _code(out.dtype), 1 if gated else 0, m, n, k, row_stats, limit=limit)
 
 
 def linear_wide_residual(x: torch.Tensor, weight: torch.Tensor, residual: torch.Tensor, norm_weight: torch.Tensor,
@@ -1926,8 +2023,10 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 WIDE_GATED_MIN_ROWS = 8192     # of the paired weight: the rule when nothing was measured
 
 
-def gated_up(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row_stats: Optional[RowStats] = None) -> None:
-    """``out[M, I] = silu(x @ gate^T) * (x @ up^T)`` with ``weight = interleave_gate_up(gate, up)``.
+def gated_up(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row_stats: Optional[RowStats] = None,
+             limit: Optional[float] = None) -> None:
+    """``out[M, I] = silu(x @ gate^T) * (x @ up^T)`` with ``weight = interleave_gate_up(gate, up)``; with ``limit`` the clamped
+    activation of :func:`silu_mul` on the two products.
     (``row_stats``: see :func:`linear_wide`; the caller has asked :func:`fold_supported` first.)
 
     Few rows of bfloat16 go through :func:`linear_wide`, which applies the activation as it stores, where that
@@ -1939,21 +2038,21 @@ def gated_up(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row_stats
     _want(out, "out", x.dtype, (m, two_i // 2))
     if row_stats is not None:
         if row_stats.per_row:
-            linear_pair(x, weight, out, gated=True, row_stats=row_stats)
+            linear_pair(x, weight, out, gated=True, row_stats=row_stats, limit=limit)
         else:
-            linear_wide(x, weight, out, gated=True, row_stats=row_stats)
+            linear_wide(x, weight, out, gated=True, row_stats=row_stats, limit=limit)
         return
     if x.dtype == torch.bfloat16 and 0 < m <= SKINNY_MAX_ROWS and _gated_choice(x, weight) == "wide":
-        linear_wide(x, weight, out, gated=True)
+        linear_wide(x, weight, out, gated=True, limit=limit)
         return
     if x.dtype == torch.bfloat16 and k % 8 == 0 and pair_preferred(x.device, m, two_i, gated=True):
         choice = _pair_or_library("gated", m, weight)
         if choice != "library":
-            linear_pair(x, weight, out, gated=True, wide=choice == "wide")    # many rows: the activation is applied as the tiles are stored
+            linear_pair(x, weight, out, gated=True, wide=choice == "wide", limit=limit)    # many rows: the activation is applied as the tiles are stored
             return
     gate_up = torch.empty((m, two_i), dtype=x.dtype, device=x.device)
     linear(x, weight, gate_up)
-    silu_mul(gate_up, out, paired=True)
+    silu_mul(gate_up, out, paired=True, limit=limit)
 
 
 def _gated_choice(x: torch.Tensor, weight: torch.Tensor) -> str:

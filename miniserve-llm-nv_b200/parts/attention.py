@@ -30,8 +30,11 @@ More options of the general form: ``bias`` (the q, k, v and output projections h
 q, k and v are added in float32 as ``kernels.qkv_prepare`` reads the heads), ``qk_norm_weight=False`` (the per-head norm of q
 and k has no weight: ``x / rms(x)``; such a norm commutes with the rotation, which turns pairs of entries and leaves a head's
 root mean square as it is, so it covers designs that norm after rotating), ``output_gate="entry"`` (the concatenated heads
-are multiplied entry by entry by ``sigmoid(W_g x)``, a gate of ``num_heads * value_dim`` rows, before the output projection) and
-``conv_taps`` (q, k and v pass a short causal convolution per channel, ``<name><conv_suffix>`` of shape ``[channels, taps]``
+are multiplied entry by entry by ``sigmoid(W_g x)``, a gate of ``num_heads * value_dim`` rows, before the output projection),
+``qk_norm="row"`` (the RMSNorm of queries and of keys runs over all their heads at once, with weights ``[n_q * head_dim]`` and
+``[n_kv * head_dim]``), ``sink="learned"`` (the sink's score is a number per query head, ``sink_name`` ``[n_q]``, not scaled) and
+``query_temperature`` (coef, every) (the queries of position p are multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)``) with
+``kernels.qkv_prepare_rows``, and ``conv_taps`` (q, k and v pass a short causal convolution per channel, ``<name><conv_suffix>`` of shape ``[channels, taps]``
 without bias, directly after the projection; the last ``taps - 1`` projected rows are the request's state, so
 ``cache_need()`` is then the pair (pages, state)).
 """
@@ -51,19 +54,20 @@ from .spec import PartSpec
 @register_mixer("attention")
 class Attention(Part):
     def __init__(self, *, prefix: str, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int,
-                 qk_norm: bool, eps: float, position: PartSpec, window: Optional[int] = None,
+                 qk_norm, eps: float, position: PartSpec, window: Optional[int] = None,
                  scale: Optional[float] = None, score_softcap: Optional[float] = None,
                  score_bias_slopes: Optional[Sequence[float]] = None,
                  q_name: str = "q_proj.weight", k_name: str = "k_proj.weight",
                  v_name: str = "v_proj.weight", o_name: str = "o_proj.weight", q_norm_name: str = "q_norm.weight",
-                 k_norm_name: str = "k_norm.weight", value_dim: Optional[int] = None, sink: bool = False,
+                 k_norm_name: str = "k_norm.weight", value_dim: Optional[int] = None, sink=False,
                  output_gate: bool = False, own_kv: bool = True, gate_name: str = "g_proj.weight",
                  values_from_keys: bool = False, bias: bool = False, bias_suffix: str = ".b", qk_norm_weight: bool = True,
-                 conv_taps: Optional[int] = None, conv_suffix: str = ".conv") -> None:
+                 conv_taps: Optional[int] = None, conv_suffix: str = ".conv", sink_name: str = "sink",
+                 query_temperature: Optional[tuple] = None) -> None:
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} key/value heads")
         general_form = bool(sink or output_gate or not own_kv or values_from_keys or (value_dim is not None and value_dim != head_dim)
-                            or bias or conv_taps or not qk_norm_weight)
+                            or bias or conv_taps or not qk_norm_weight or qk_norm == "row" or query_temperature is not None)
         if general_form and 1 <= head_dim <= kernels.MAX_HEAD_DIM:
             pass            # (the general form's kernels take odd head sizes too; the rotation checks its own size)
         elif head_dim % 2 or not 2 <= head_dim <= kernels.MAX_HEAD_DIM:
@@ -72,7 +76,17 @@ class Attention(Part):
             raise ValueError(f"head size {head_dim} is not an even number in 2..{kernels.MAX_HEAD_DIM}")
         self.prefix = prefix
         self.hidden_size, self.num_heads, self.num_kv_heads, self.head_dim = hidden_size, num_heads, num_kv_heads, head_dim
+        if qk_norm not in (False, True, "head", "row") or sink not in (False, True, "learned"):
+            raise ValueError(f"qk_norm is False, 'head' (True) or 'row' and sink False, True or 'learned', not {qk_norm!r} and {sink!r}")
         self.qk_norm, self.eps = bool(qk_norm), float(eps)
+        self.norm_over_row = qk_norm == "row"
+        self.query_temperature = None if query_temperature is None else (float(query_temperature[0]), float(query_temperature[1]))
+        # queries and keys prepared a whole row at a time (a norm over all heads, a temperature of the queries)
+        self.prepare_rows = self.norm_over_row or self.query_temperature is not None
+        if self.prepare_rows and (not own_kv or values_from_keys or bias or (qk_norm and not self.norm_over_row) or not qk_norm_weight):
+            raise ValueError("a norm over the whole row and a query temperature go with the layer's own keys and values, without "
+                             "biases and without a norm per head")
+        self.learned_sink, self.sink_scores = sink == "learned", None
         self.window = window
         self.scale = float(scale) if scale is not None else head_dim ** -0.5
         self.score_softcap = float(score_softcap) if score_softcap else None
@@ -99,11 +113,12 @@ class Attention(Part):
         if self.values_from_keys and (self.value_dim != head_dim or not self.own_kv):
             raise ValueError("values_from_keys: the values are the layer's own keys, so both have the same size")
         self.general = (self.sink or self.output_gate or not self.own_kv or self.values_from_keys or self.value_dim != head_dim
-                        or self.bias or self.conv_taps is not None or not self.qk_norm_weight)
+                        or self.bias or self.conv_taps is not None or not self.qk_norm_weight or self.prepare_rows)
         if self.general and (self.score_softcap or self.score_bias_slopes is not None):
             raise ValueError("score modifiers are not implemented together with value_dim, sink, output_gate or own_kv=False")
         self.names = dict(q=prefix + q_name, k=prefix + k_name, v=prefix + v_name, o=prefix + o_name,
-                          q_norm=prefix + q_norm_name, k_norm=prefix + k_norm_name, g=prefix + gate_name)
+                          q_norm=prefix + q_norm_name, k_norm=prefix + k_norm_name, g=prefix + gate_name,
+                          sink=prefix + sink_name)
         for key in ("q", "k", "v", "o"):
             self.names[key + "_b"] = self.names[key] + bias_suffix
             self.names[key + "_conv"] = self.names[key] + conv_suffix
@@ -133,9 +148,11 @@ class Attention(Part):
             if not self.values_from_keys:
                 specs.append(ParamSpec(self.names["v"], (self.num_kv_heads * dv, h)))
         if self.qk_norm and self.qk_norm_weight:
-            specs.append(ParamSpec(self.names["q_norm"], (d,), "vector"))
+            specs.append(ParamSpec(self.names["q_norm"], (self.num_heads * d if self.norm_over_row else d,), "vector"))
             if self.own_kv:
-                specs.append(ParamSpec(self.names["k_norm"], (d,), "vector"))
+                specs.append(ParamSpec(self.names["k_norm"], (self.num_kv_heads * d if self.norm_over_row else d,), "vector"))
+        if self.learned_sink:
+            specs.append(ParamSpec(self.names["sink"], (self.num_heads,), "vector"))
         if self.output_gate:
             specs.append(ParamSpec(self.names["g"], (self.gate_rows, h)))
         specs.append(ParamSpec(self.names["o"], (h, self.num_heads * dv)))
@@ -162,6 +179,8 @@ class Attention(Part):
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         n = self.names
         self.o_weight = tensors[n["o"]]
+        if self.learned_sink:
+            self.sink_scores = tensors[n["sink"]].float().contiguous()
         if self.general:
             pieces = [tensors[n["q"]]] + ([tensors[n["k"]]] if self.own_kv else [])
             if self.own_kv and not self.values_from_keys:
@@ -277,15 +296,20 @@ class Attention(Part):
                                 ctx.max_query_len, heads, activation="none", in_bias=self.in_bias)
         cos_sin, rotary_dim, interleaved = self.position.fused_args(ctx)
         q = ctx.buffer("attention.q", (n, n_q, d), x.dtype)
-        kernels.qkv_prepare(heads, 0, self.k_col, self.v_col, n_q, n_kv, d, dv, cache.slots, self.q_norm_weight,
-                            self.k_norm_weight, self.eps, cos_sin, rotary_dim, cache.key_pool, cache.value_pool, q,
-                            interleaved=interleaved, bias=self.in_bias if state is None else None)
+        if self.prepare_rows:
+            kernels.qkv_prepare_rows(heads, 0, self.k_col, self.v_col, n_q, n_kv, d, dv, cache.slots, self.q_norm_weight,
+                                     self.k_norm_weight, self.eps, cos_sin, rotary_dim, cache.key_pool, cache.value_pool, q,
+                                     interleaved=interleaved, positions=ctx.positions, temperature=self.query_temperature)
+        else:
+            kernels.qkv_prepare(heads, 0, self.k_col, self.v_col, n_q, n_kv, d, dv, cache.slots, self.q_norm_weight,
+                                self.k_norm_weight, self.eps, cos_sin, rotary_dim, cache.key_pool, cache.value_pool, q,
+                                interleaved=interleaved, bias=self.in_bias if state is None else None)
         attended = ctx.buffer("attention.attended", (n, n_q, dv), x.dtype)
         per_head = self.output_gate and not self.gate_per_entry
         kernels.paged_attention(q, cache.key_pool, cache.value_pool, cache.block_tables, ctx.request_of_token,
                                 ctx.positions, ctx.query_start, ctx.context_lens, ctx.max_query_len,
                                 ctx.max_context_len, self.scale, self.window, attended, ctx.host_query_start or None,
-                                sink=self.sink, gate=proj if per_head else None, gate_col=max(self.gate_col, 0))
+                                sink=self.sink_scores if self.learned_sink else self.sink, gate=proj if per_head else None, gate_col=max(self.gate_col, 0))
         if self.gate_per_entry:
             kernels.sigmoid_gate_mul(attended.view(n, n_q * dv), proj, self.gate_col, attended.view(n, n_q * dv))
         out = ctx.buffer("attention.out", (n, self.hidden_size), x.dtype)

@@ -16,12 +16,14 @@ mixer           ``forward(x, ctx, cache) -> y``; ``cache_need()`` says what ``ca
                 mixer made of several: ``cache`` is then the tuple of their views)
 feed_forward    ``forward(x, ctx) -> y``
 block           ``forward(residual, delta, ctx, cache) -> delta``: arranges the four above
+transition      ``remember(residual, ctx)`` once a step behind the embedding, ``enter(residual, pending, ctx, number)
+                -> pending`` before the layer runs that name it: what happens to the stream between two layers
 embedding       ``add(residual, ctx, cache)``: adds rows of a table of its own to the token embeddings in the
                 float32 stream; ``cache_need()`` as for a mixer (a state that a sequence carries, or None)
 ==============  ==========================================================================
 
 A new part is a class registered under a name with ``register_norm`` / ``register_position``
-/ ``register_mixer`` / ``register_feed_forward`` / ``register_block``; an architecture then
+/ ``register_mixer`` / ``register_feed_forward`` / ``register_block`` / ``register_transition``; an architecture then
 names it in its :class:`~.spec.PartSpec`.
 
 Optional, for speed in steps of few rows: a norm between two matrix products can be *folded* into
@@ -166,6 +168,14 @@ class ChannelScaled:
 
 
 @dataclass
+class StreamVector:
+    """What a transition hands on where one vector (float32 ``[hidden]``) is still to be added to every row of the stream: the
+    norm that reads the stream next adds it in float32."""
+
+    vector: torch.Tensor
+
+
+@dataclass
 class FoldedInput:
     """What a part receives as ``x`` where the norm before it was folded: ``x = residual * norm weight`` and the
     statistics that its first product completes the norm with (``kernels.RowStats``)."""
@@ -212,6 +222,7 @@ POSITIONS = Registry("position")
 MIXERS = Registry("mixer")
 FEED_FORWARDS = Registry("feed_forward")
 BLOCKS = Registry("block")
+TRANSITIONS = Registry("transition")
 
 register_norm = NORMS.register
 register_embedding = EMBEDDINGS.register
@@ -219,3 +230,4 @@ register_position = POSITIONS.register
 register_mixer = MIXERS.register
 register_feed_forward = FEED_FORWARDS.register
 register_block = BLOCKS.register
+register_transition = TRANSITIONS.register

@@ -1,6 +1,7 @@
 """Block arrangements.  ``pre_norm``: ``h += mixer(norm(h)); h += feed_forward(norm(h))``
 (miniserve/model/qwen3.py:336-346).  ``parallel``: one norm whose output both sublayers read,
 ``h += mixer(norm(h)) + feed_forward(norm(h))``; a layer without a feed-forward is ``h += mixer(norm(h))``.
+``parallel_two_norms``: the same with a norm of its own for each sublayer, ``h += mixer(norm_1(h)) + feed_forward(norm_2(h))``.
 ``sandwich``: a norm on both sides of each sublayer, ``h += post(mixer(norm(h))); h += post(feed_forward(norm(h)))``.
 ``scaled_pre_norm``: ``pre_norm`` where what a sublayer adds is multiplied by a constant and, channel by channel, by a vector
 of the layer (a layer scale): ``h += m * s1 * mixer(norm(h)); h += m * s2 * feed_forward(norm(h))``.
@@ -25,11 +26,11 @@ from typing import Any, Optional, Union
 import torch
 
 from .. import kernels
-from .base import ChannelScaled, FoldedInput, NormFold, ParamSpec, Part, PostNormed, ResidualAdd, register_block
+from .base import ChannelScaled, FoldedInput, NormFold, ParamSpec, Part, PostNormed, ResidualAdd, StreamVector, register_block
 from .context import StepContext
 
 # what a block hands on: nothing, an output still to add (or two, whose float32 sum is to be added), or a folded input
-Pending = Union[None, torch.Tensor, tuple, FoldedInput, PostNormed, ChannelScaled]
+Pending = Union[None, torch.Tensor, tuple, FoldedInput, PostNormed, ChannelScaled, StreamVector]
 
 
 def fold_between(producer, norm, consumer, ctx: StepContext) -> Optional[tuple]:
@@ -122,6 +123,41 @@ class ParallelBlock:
         if self.feed_forward is None:
             return mixed
         return mixed, self.feed_forward.forward(normed, ctx)
+
+
+@register_block("parallel_two_norms")
+class ParallelTwoNormsBlock:
+    """``x <- x + (mixer(norm_1(x)) + feed_forward(norm_2(x)))``: both sublayers read the same stream, each through a norm of its
+    own; a layer without a feed-forward is ``x <- x + mixer(norm_1(x))``.  Norms that share their statistics (two layer norms)
+    run as one kernel that reads the stream once.  The outputs are handed on as by :class:`ParallelBlock`.
+    """
+
+    def __init__(self, *, mixer, feed_forward, mixer_norm, feed_forward_norm=None) -> None:
+        if (feed_forward is None) != (feed_forward_norm is None):
+            raise ValueError("a parallel block with two norms has a feed-forward with its norm, or neither")
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
+
+    def parts(self):
+        return [part for part in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if part is not None]
+
+    def forward(self, residual: torch.Tensor, pending: Pending, ctx: StepContext, cache: Any) -> Pending:
+        if isinstance(pending, FoldedInput):
+            raise TypeError("a parallel block takes its input from its own norms")
+        # (buffers of their own: the pending outputs of the layer before live in the parts' buffers until they are added here)
+        normed = ctx.buffer("parallel.normed", tuple(residual.shape), ctx.dtype)
+        if self.feed_forward is None:
+            self.mixer_norm.add_and_norm(residual, pending, normed)
+            return self.mixer.forward(normed, ctx, cache)
+        normed_2 = ctx.buffer("parallel.normed_2", tuple(residual.shape), ctx.dtype)
+        shares = getattr(self.mixer_norm, "shares_statistics_with", None)
+        if shares is not None and shares(self.feed_forward_norm):
+            self.mixer_norm.add_and_norm_both(residual, pending, normed, self.feed_forward_norm, normed_2)
+        else:
+            self.mixer_norm.add_and_norm(residual, pending, normed)
+            self.feed_forward_norm.add_and_norm(residual, None, normed_2)
+        mixed = self.mixer.forward(normed, ctx, cache)
+        return mixed, self.feed_forward.forward(normed_2, ctx)
 
 
 @register_block("sandwich")

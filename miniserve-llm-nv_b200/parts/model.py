@@ -13,7 +13,7 @@ from typing import Any, Optional, Union
 import torch
 
 from .. import kernels
-from .base import BLOCKS, EMBEDDINGS, FEED_FORWARDS, MIXERS, NORMS, PagedKVNeed, PagedLatentNeed, ParamSpec, StateNeed
+from .base import BLOCKS, EMBEDDINGS, FEED_FORWARDS, MIXERS, NORMS, TRANSITIONS, PagedKVNeed, PagedLatentNeed, ParamSpec, StateNeed
 from .context import StepContext
 from .spec import ModelSpec
 
@@ -50,11 +50,14 @@ class DecoderModel:
                                             mixer_norm=mixer_norm, feed_forward_norm=feed_forward_norm, **post))
         self.final_norm = NORMS.build(spec.final_norm)
         self.extra_embeddings = [EMBEDDINGS.build(part) for part in spec.extra_embeddings]
+        self.transitions = [TRANSITIONS.build(part) for part in spec.transitions]
         for index, run in enumerate(spec.order):
             if not 0 <= run.layer < len(self.blocks):
                 raise ValueError(f"order[{index}] names layer {run.layer}, the model has {len(self.blocks)}")
             if run.cache_of is not None and not 0 <= run.cache_of < index:
                 raise ValueError(f"order[{index}] reads the cache of entry {run.cache_of}, which does not come before it")
+            if run.enters is not None and not 0 <= run.enters[0] < len(self.transitions):
+                raise ValueError(f"order[{index}] enters through transition {run.enters[0]}, the model has {len(self.transitions)}")
         self.cache_groups, self.run_caches, self.embedding_caches = self._plan_caches()
         self.embedding: Optional[torch.Tensor] = None
         self.output_weight: Optional[torch.Tensor] = None
@@ -64,6 +67,7 @@ class DecoderModel:
         yield from self.extra_embeddings
         for block in self.blocks:
             yield from block.parts()
+        yield from self.transitions
         yield self.final_norm
 
     def param_specs(self) -> list[ParamSpec]:
@@ -136,13 +140,18 @@ class DecoderModel:
         kernels.embedding(ctx.token_ids, self.embedding, residual, spec.embedding_scale)
         for part, plan in zip(self.extra_embeddings, self.embedding_caches):
             part.add(residual, ctx, None if plan is None else storage.run_view(plan, ctx))
+        for transition in self.transitions:
+            transition.remember(residual, ctx)
         delta = None            # what a block hands to the next: see parts.block
         for index, run in enumerate(spec.order):
             plan = self.run_caches[index]
             cache = None if plan is None else storage.run_view(plan, ctx)
             block = self.blocks[run.layer]
+            if run.enters is not None:
+                delta = self.transitions[run.enters[0]].enter(residual, delta, ctx, run.enters[1])
             if getattr(block, "takes_next_block", False):
-                following = self.blocks[spec.order[index + 1].layer] if index + 1 < len(spec.order) else None
+                after = spec.order[index + 1] if index + 1 < len(spec.order) else None
+                following = None if after is None or after.enters is not None else self.blocks[after.layer]
                 delta = block.forward(residual, delta, ctx, cache, following)
             else:
                 delta = block.forward(residual, delta, ctx, cache)

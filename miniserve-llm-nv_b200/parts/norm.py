@@ -2,7 +2,8 @@
 (miniserve/model/layers.py:30-34), fused with the residual add that precedes it.  ``one_plus``: the stored weight
 lies around zero and stands for ``1 + weight`` (added once, in float32, when the weight is loaded).  ``identity``: no norm
 at all, for blocks whose sublayers read the residual stream itself: what is pending is added and the stream is handed on in
-the compute type."""
+the compute type.  ``layer``: layer norm with weight and bias, ``weight * (x - mean) / sqrt(mean((x - mean)^2) + eps) + bias``;
+two of them that read the same stream run as one kernel (``add_and_norm_both``)."""
 
 from __future__ import annotations
 
@@ -11,7 +12,7 @@ from typing import Optional
 import torch
 
 from .. import kernels
-from .base import ChannelScaled, ParamSpec, Part, PostNormed, register_norm
+from .base import ChannelScaled, ParamSpec, Part, PostNormed, StreamVector, register_norm
 
 
 @register_norm("rms")
@@ -47,6 +48,9 @@ class RMSNorm(Part):
             # the output of the sublayer before is multiplied channel by channel (in float32) on its way into the stream
             kernels.postnorm_add_rmsnorm(residual, delta.x, delta.weight, 0.0, self.weight, self.eps, out, rows, post_norm=False)
             return out
+        if isinstance(delta, StreamVector):
+            kernels.add_bias(residual, delta.vector)
+            delta = None
         second = None
         if isinstance(delta, tuple):
             delta, second = delta
@@ -74,6 +78,9 @@ class IdentityNorm(Part):
 
     def add_and_norm(self, residual: torch.Tensor, delta, out: torch.Tensor,
                      rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if isinstance(delta, StreamVector):
+            kernels.add_bias(residual, delta.vector)
+            delta = None
         if delta is None:
             kernels.postnorm_add_rmsnorm(residual, None, None, 0.0, None, 0.0, out, rows)
         elif isinstance(delta, PostNormed):
@@ -81,3 +88,48 @@ class IdentityNorm(Part):
         else:
             raise TypeError("the identity norm adds nothing, or an output that passes a norm of its own")
         return out
+
+
+@register_norm("layer")
+class LayerNorm(Part):
+    """Layer norm with weight and bias (``name`` and ``name + bias_suffix``), statistics in float32."""
+
+    def __init__(self, *, name: str, size: int, eps: float, prefix: str = "", bias_suffix: str = ".b") -> None:
+        self.name, self.bias_name, self.size, self.eps = prefix + name, prefix + name + bias_suffix, size, float(eps)
+        self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+
+    def param_specs(self) -> list[ParamSpec]:
+        return [ParamSpec(self.name, (self.size,), "vector"), ParamSpec(self.bias_name, (self.size,), "vector")]
+
+    def load(self, tensors: dict[str, torch.Tensor]) -> None:
+        self.weight, self.bias = tensors[self.name], tensors[self.bias_name]
+        if self.weight.dtype != self.bias.dtype:
+            self.weight, self.bias = self.weight.float(), self.bias.float()
+
+    @staticmethod
+    def _pending(delta) -> tuple:
+        """(first output, second output, vector) of what is still to be added to the stream."""
+        if isinstance(delta, StreamVector):
+            return None, None, delta.vector
+        if delta is None or isinstance(delta, torch.Tensor):
+            return delta, None, None
+        if isinstance(delta, tuple):
+            return delta[0], delta[1], None
+        raise TypeError(f"the layer norm adds outputs or a vector, not {type(delta).__name__}")
+
+    def add_and_norm(self, residual: torch.Tensor, delta, out: torch.Tensor,
+                     rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``residual += delta`` (float32, in place), ``out = norm(residual)``, as :meth:`RMSNorm.add_and_norm`."""
+        first, second, vector = self._pending(delta)
+        kernels.add_layernorm(residual, first, self.weight, self.bias, self.eps, out, rows, second, vector)
+        return out
+
+    def shares_statistics_with(self, other) -> bool:
+        """Whether :meth:`add_and_norm_both` can run this norm and ``other`` on the same stream in one kernel."""
+        return isinstance(other, LayerNorm) and other.eps == self.eps and other.weight.dtype == self.weight.dtype
+
+    def add_and_norm_both(self, residual: torch.Tensor, delta, out: torch.Tensor, other: "LayerNorm", other_out: torch.Tensor) -> None:
+        first, second, vector = self._pending(delta)
+        kernels.add_layernorm(residual, first, self.weight, self.bias, self.eps, out, None, second, vector, other.weight, other.bias,
+                              other_out)

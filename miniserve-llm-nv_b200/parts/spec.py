@@ -43,11 +43,13 @@ class LayerRun:
 
     ``cache_of`` is ``None`` when the run keeps a cache of its own (if its mixer needs one);
     otherwise it is the index of an earlier entry of the order whose cache this run reads
-    without writing to it.
+    without writing to it.  ``enters`` is ``None`` or a pair ``(transition, number)``: before this run the stream goes
+    through ``ModelSpec.transitions[transition]``, for the ``number``-th time of the step (the first is 0).
     """
 
     layer: int
     cache_of: Optional[int] = None
+    enters: Optional[tuple] = None
 
 
 @dataclass(frozen=True)
@@ -77,3 +79,5 @@ class ModelSpec:
     # Parts of the embedding family whose rows are added to the (scaled) token embeddings, each with a table of its own
     # and, where it looks back along the sequence, a state that the request carries.
     extra_embeddings: Sequence[PartSpec] = ()
+    # Parts of the transition family: what happens to the stream between two layers, where ``LayerRun.enters`` says so.
+    transitions: Sequence[PartSpec] = ()

@@ -96,7 +96,7 @@ def qk_norm_rope_append(qkv, slots, q_weight, k_weight, eps, cos_sin, rotary_dim
         v_pool[page, :, offset, :] = v[token].to(v_pool.dtype)
 
 
-def silu_mul(gate_up, out, paired=False, bias=None):
+def silu_mul(gate_up, out, paired=False, bias=None, limit=None):
     n, inter = out.shape
     if bias is not None:
         gate_up = gate_up.double() + bias.double()
@@ -105,7 +105,7 @@ def silu_mul(gate_up, out, paired=False, bias=None):
         g, u = blocks[:, :, 0].reshape(n, inter).double(), blocks[:, :, 1].reshape(n, inter).double()
     else:
         g, u = gate_up[:, :inter].double(), gate_up[:, inter:].double()
-    out.copy_((g * torch.sigmoid(g) * u).to(out.dtype))
+    out.copy_((clamped_glu_values(g, u, limit) if limit else g * torch.sigmoid(g) * u).to(out.dtype))
 
 
 def _row_factor(row_stats, size):
@@ -114,11 +114,11 @@ def _row_factor(row_stats, size):
     return 1.0 / torch.sqrt(total / size + row_stats.eps)
 
 
-def gated_up(x, weight, out, row_stats=None):
+def gated_up(x, weight, out, row_stats=None, limit=None):
     gate_up = x.double() @ weight.double().T
     if row_stats is not None:
         gate_up = gate_up * _row_factor(row_stats, x.shape[1])[:x.shape[0], None]
-    silu_mul(gate_up.to(x.dtype), out, paired=True)
+    silu_mul(gate_up.to(x.dtype), out, paired=True, limit=limit)
 
 
 FOLD_BLOCKS = 3     # the plain stand-in leaves its sums of squares in this many rows, as a kernel of three blocks would
@@ -164,7 +164,11 @@ def paged_attention(q, k_pool, v_pool, block_tables, request_of_token, positions
                 scores = softcap * torch.tanh(scores / softcap)
             if bias_slopes is not None:
                 scores = scores + float(bias_slopes[head]) * (keys - pos).double()
-            if sink:        # one more term exp(0) in the denominator: a key of score 0 without a value
+            if isinstance(sink, torch.Tensor):      # one more term exp(sink[head]) in the denominator
+                top = torch.maximum(scores.max(), sink[head].double())
+                e = torch.exp(scores - top)
+                p = e / (e.sum() + torch.exp(sink[head].double() - top))
+            elif sink:        # one more term exp(0) in the denominator: a key of score 0 without a value
                 top = torch.clamp(scores.max(), min=0.0)
                 e = torch.exp(scores - top)
                 p = e / (e.sum() + torch.exp(-top))
@@ -206,7 +210,8 @@ def sample(logits, records, slot_of_row, draw_index, out):
 # --------------------------------------------------------------------------- latent attention
 
 
-def latent_prepare(proj, q_col, dkv_col, heads, dim, rot, rank, slots, norm_weight, eps, cos_sin, rot_dims, cache, q_full):
+def latent_prepare(proj, q_col, dkv_col, heads, dim, rot, rank, slots, norm_weight, eps, cos_sin, rot_dims, cache, q_full,
+                   interleaved=False):
     n = proj.shape[0]
     p = proj.double()
 
@@ -217,8 +222,9 @@ def latent_prepare(proj, q_col, dkv_col, heads, dim, rot, rank, slots, norm_weig
         shape = [n] + [1] * (x.dim() - 2) + [half]
         cos, sin = cos_sin[..., 0].double().view(shape), cos_sin[..., 1].double().view(shape)
         out = x.clone()
-        u, v = x[..., :half], x[..., half:rot_dims]
-        out[..., :half], out[..., half:rot_dims] = u * cos - v * sin, v * cos + u * sin
+        first, second = (slice(0, rot_dims, 2), slice(1, rot_dims, 2)) if interleaved else (slice(0, half), slice(half, rot_dims))
+        u, v = x[..., first], x[..., second]
+        out[..., first], out[..., second] = u * cos - v * sin, v * cos + u * sin
         return out
 
     q = p[:, q_col:q_col + heads * (dim + rot)].view(n, heads, dim + rot)
@@ -394,6 +400,56 @@ def qkv_prepare(proj, q_col, k_col, v_col, n_q, n_kv, head_dim, value_dim, slots
             continue
         k_pool[slot // page_size, :, slot % page_size, :] = k[token].to(k_pool.dtype)
         v_pool[slot // page_size, :, slot % page_size, :] = v[token].to(v_pool.dtype)
+
+
+def qkv_prepare_rows(proj, q_col, k_col, v_col, n_q, n_kv, head_dim, value_dim, slots, q_weight, k_weight, eps, cos_sin, rotary_dim,
+                     k_pool, v_pool, q_out, interleaved=False, positions=None, temperature=None):
+    n = proj.shape[0]
+
+    def heads(col, count, weight):
+        x = proj[:, col:col + count * head_dim].double()
+        if weight is not None:
+            x = weight.double() * (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps))
+        x = x.view(n, count, head_dim)
+        return x if cos_sin is None else rotate(x, cos_sin, rotary_dim, interleaved)
+
+    q = heads(q_col, n_q, q_weight)
+    if temperature is not None:
+        coef, every = temperature
+        q = q * (1.0 + coef * torch.log(torch.floor((positions.double() + 1.0) / every) + 1.0)).view(n, 1, 1)
+    q_out.copy_(q.to(q_out.dtype))
+    k, v = heads(k_col, n_kv, k_weight), proj[:, v_col:v_col + n_kv * value_dim].view(n, n_kv, value_dim)
+    page_size = k_pool.shape[2]
+    for token in range(n):
+        slot = int(slots[token])
+        if slot >= 0:
+            k_pool[slot // page_size, :, slot % page_size, :] = k[token].to(k_pool.dtype)
+            v_pool[slot // page_size, :, slot % page_size, :] = v[token].to(v_pool.dtype)
+
+
+def add_layernorm(residual, delta, weight, bias, eps, out, rows=None, delta2=None, vector=None, weight2=None, bias2=None, out2=None):
+    add = torch.zeros_like(residual, dtype=torch.float64)
+    for piece in (delta, delta2, vector):
+        if piece is not None:
+            add = add + piece.double()
+    if rows is None:
+        residual += add.to(residual.dtype)
+        x = residual.double()
+    else:
+        x = (residual.double() + add)[rows.long()]
+    x = x - x.mean(-1, keepdim=True)
+    y = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+    out.copy_((weight.double() * y + bias.double()).to(out.dtype))
+    if out2 is not None:
+        out2.copy_((weight2.double() * y + bias2.double()).to(out2.dtype))
+
+
+def stream_to_columns(residual, delta, out, col, delta2=None):
+    x = residual.double()
+    for piece in (delta, delta2):
+        if piece is not None:
+            x = x + piece.double()
+    out[:, col:col + residual.shape[1]] = x.to(out.dtype)
 
 
 # --------------------------------------------------------------------------- state-space mixer
@@ -660,7 +716,7 @@ def install(monkeypatch) -> None:
                  "selective_scan", "gated_group_norm", "causal_conv", "add_bias", "scaled_sum", "small_linear_f32",
                  "unit_norm_heads", "exponential_gates", "decay_gates", "matrix_scan", "head_norm_gate", "gated_recurrence_scan",
                  "low_rank_expand", "channel_decays", "normed_sum", "sigmoid_gate_mul", "differential_combine", "token_shift",
-                 "pair_embedding"):
+                 "pair_embedding", "qkv_prepare_rows", "add_layernorm", "stream_to_columns"):
         monkeypatch.setattr(kernels, name, globals()[name])
     monkeypatch.setattr(kernels, "attention_kernels", lambda *sizes: {"decode": "plain", "prompt": "plain"})
     monkeypatch.setattr(kernels, "latent_attention_kernels", lambda *sizes: {"decode": "plain", "prompt": "plain"})
