@@ -481,9 +481,10 @@ def _latent(heads, dim, rot, vdim, rank):
 
 
 def _vesidra(width, layers, mixer, dense_ff, experts, top, expert_ff, shared_ff, vocab):
+    """``experts`` 0: every layer has the gated MLP; else every other layer has experts."""
     entries = []
     for index in range(layers):
-        mlp = dict(kind="dense", ff=dense_ff) if index % 2 == 0 else dict(
+        mlp = dict(kind="dense", ff=dense_ff) if index % 2 == 0 or not experts else dict(
             kind="moe", expert=dict(ff=expert_ff), router=dict(experts=experts, top=top), shared=dict(ff=shared_ff))
         entries.append(dict(type="latent_attention", mixer=mixer, mlp=mlp))
     return dict(architecture="Vesidra", vocab=vocab, width=width, embedding=dict(scale=float(width) ** 0.5), norm=dict(eps=1e-6),
@@ -541,6 +542,20 @@ def _bafavik(width, left, linear, differential, delta, ff, vocab):
                 layers=[dict(pair, mlp=mlp), dict(diff, mlp=mlp), dict(pair_2, mlp=mlp), dict(pair, mlp=mlp)])
 
 
+def _venarax(width, latent, window, sink, ff, vocab):
+    """Four layers (latent attention behind a window, attention with sinks, the same again), the two in the middle run twice: six
+    layer runs in all, and two mixes with the embedding output."""
+    heads, dim, rot, vdim, rank = latent
+    windowed = dict(type="latent_attention", mixer=dict(heads=heads, dim=dim, rot_dim=rot, vdim=vdim, kv_rank=rank, scale=(dim + rot) ** -0.5,
+                                                        rot=dict(base=10000.0, dims=rot), mask=dict(size=window)))
+    heads, kv_heads, dim, vdim = sink
+    full = dict(type="attention", mixer=dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=dim ** -0.5,
+                                             q_temp=dict(coef=0.1, every=8192)))
+    mlp = dict(kind="dense", ff=ff, limit=7.0)
+    return dict(architecture="Venarax", vocab=vocab, width=width, norm=dict(eps=1e-6), loop=dict(start=1, stop=3, times=2),
+                layers=[dict(mixer, mlp=mlp) for mixer in (windowed, full, windowed, full)])
+
+
 # Layer sizes that resemble real models' (random weights, four layers each: two with a gated MLP, two with experts), and
 # the Qwen3 layers of equal width, head count and inner size beside them.
 DESIGN_SIZES = {
@@ -581,11 +596,21 @@ DESIGN_SIZES = {
     "pairs-lite": dict(bafavik=_bafavik(2048, (32, 8, 64, 64), (32, 64, 64), (32, 8, 64, 64, 512), (32, 16, 64, 64, 32), 10944, 32000),
                        kivurax=_kivurax(2048, (16, 64, 128), (32, 16, 64, 64), (32, 8, 64, 512), (2560, 20), 10944, 60, 6, 1408, 32000),
                        qwen3=dict(hidden_size=2048, intermediate_size=10944, num_attention_heads=32, num_key_value_heads=8, head_dim=64)),
+    # Venarax: latent 256 + 32 with sixteen heads of 64 + 32 behind a window of 1,024, and sixteen heads of 128 over four key heads
+    # with sinks; feed-forward 6,144; six layer runs.  Beside it six layers of Vesidra (the closest design: parallel blocks of latent
+    # attention and a gated feed-forward, here without experts) and six of Qwen3
+    "windowed-small": dict(venarax=_venarax(2048, (16, 64, 32, 64, 256), 1024, (16, 4, 128, 128), 6144, 32000),
+                           vesidra=_vesidra(2048, 6, _latent(16, 64, 32, 64, 256), 6144, 0, 0, 0, 0, 32000), depth=6,
+                           qwen3=dict(hidden_size=2048, intermediate_size=6144, num_attention_heads=16, num_key_value_heads=4, head_dim=128)),
+    # latent 512 + 64 with sixteen heads of 128 + 64 behind a window of 512, 32 heads of 64 over eight key heads, feed-forward 10,944
+    "windowed-lite": dict(venarax=_venarax(2048, (16, 128, 64, 128, 512), 512, (32, 8, 64, 64), 10944, 32000),
+                          vesidra=_vesidra(2048, 6, _latent(16, 128, 64, 128, 512), 10944, 0, 0, 0, 0, 32000), depth=6,
+                          qwen3=dict(hidden_size=2048, intermediate_size=10944, num_attention_heads=32, num_key_value_heads=8, head_dim=64)),
 }
 
 
 def designs_workload(args) -> int:
-    """``--workload designs``: prompt and decode throughput of Vesidra, Zozezen, Kivurax and Bafavik at sizes that resemble real models' layers, beside
+    """``--workload designs``: prompt and decode throughput of Vesidra, Zozezen, Kivurax, Bafavik and Venarax at sizes that resemble real models' layers, beside
     the Qwen3 decoder at equal width, depth, head count and inner size; one JSON line per size and design, with each
     step's kernels (device time by kernel, from the framework profiler) so that like kernels can be set side by side."""
     import torch
@@ -602,12 +627,12 @@ def designs_workload(args) -> int:
     for size_name, pair in DESIGN_SIZES.items():
         if args.design_size and size_name != args.design_size:
             continue
-        own = {name: config for name, config in pair.items() if name != "qwen3"}
-        layers = len(next(iter(own.values()))["layers"])
+        own = {name: config for name, config in pair.items() if name not in ("qwen3", "depth")}
+        layers = pair.get("depth") or len(next(iter(own.values()))["layers"])
         vocab = next(iter(own.values()))["vocab"]
         configs = dict(own, qwen3=dict(MODEL, **pair["qwen3"], num_hidden_layers=layers, vocab_size=vocab, tie_word_embeddings=True))
         for design, config in configs.items():
-            # (a model with per-request state cannot be cut back between the timed blocks: its contexts grow through all of them)
+            # (a model with per-request state or a window cannot be cut back between the timed blocks: its contexts grow through all of them)
             room = context + 8 * steps + warmup + 8
             pages = batch * ((room + PAGE_SIZE - 1) // PAGE_SIZE) + prompt_tokens // PAGE_SIZE + 8
             runtime = build_runtime(None, EngineConfig(
@@ -680,7 +705,7 @@ def designs_workload(args) -> int:
                     manager.commit(reservation)
 
             def rewind() -> None:
-                if manager.state_needs:
+                if manager.state_needs or any(not need.keeps_all for need in manager.paged_needs):
                     return
                 for rid in ids:
                     manager.truncate(rid, context)
@@ -736,7 +761,7 @@ def main() -> int:
                         help="fewer layers than the model has (named in the output); for quick checks only")
     parser.add_argument("--skip-points", action="store_true")
     parser.add_argument("--workload", choices=("default", "mixed", "sweep", "designs"), default="default",
-                        help="designs: Vesidra, Zozezen, Kivurax and Bafavik beside Qwen3 at equal layer sizes (prompt and decode throughput, kernels by time)")
+                        help="designs: Vesidra, Zozezen, Kivurax, Bafavik and Venarax beside Qwen3 at equal layer sizes (prompt and decode throughput, kernels by time)")
     parser.add_argument("--design-size", choices=sorted(DESIGN_SIZES), default=None, help="with --workload designs: one size only")
     parser.add_argument("--sweep-prompt", type=int, default=1024)
     parser.add_argument("--sweep-new", type=int, default=128)
