@@ -517,21 +517,33 @@ MS_EXPORT int ms_latent_attention_mma_supports(int rank, int rot, int heads) {
   return rank_ok && rot >= 0 && rot % 16 == 0 && rank + rot <= 1024 && heads >= 1 && heads <= 65535 ? 1 : 0;
 }
 
-// How many ranges the keys of a step are cut into: 1 for steps with prompt portions; for steps of single tokens enough
-// that the blocks fill the multiprocessors about four times, at most one range per two key tiles of the longest
-// context (`max_context_len`, an upper bound), and at most 32 (16 for a latent of 512: the merge that takes more
-// than 16 ranges holds sixteen partial results per thread).
+// How many ranges the keys of a step are cut into: 1 for steps with prompt portions; for steps of single tokens the number whose
+// blocks, in rounds of as many as the multiprocessors hold (their shared memory decides), take the fewest tile times: a round
+// lasts as long as one block's tiles and what a block costs before its first tile (about three tiles), and every range is
+// one more partial result to merge (an eighth of a tile).  `max_context_len`: an upper bound on the keys a token sees; at most
+// one range per two key tiles, and at most 32 ranges (16 for a latent of 512: the merge that takes more than 16 ranges holds
+// sixteen partial results per thread).
 MS_EXPORT int ms_latent_attention_mma_splits(int rank, int rot, int heads, int n_requests, int max_query_len,
                                              int max_context_len) {
   if (max_query_len != 1 || n_requests <= 0) return 1;
   const int row_tiles = (heads + 15) / 16;
-  const int blocks = n_requests * row_tiles;
-  int splits = (4 * latent_sm_count() + blocks - 1) / blocks;
+  const long long rows = (long long)n_requests * row_tiles;
   const int by_keys = (max_context_len + 2 * LBN - 1) / (2 * LBN);
-  const int most = rank > 256 ? 16 : 32;
-  if (splits > by_keys) splits = by_keys;
-  if (splits > most) splits = most;
-  return splits < 1 ? 1 : splits;
+  const int most = min(rank > 256 ? 16 : 32, by_keys);
+  const int tiles = max_context_len / LBN + 1;
+  const int smem = (16 + 4 * LBN) * (rank + rot + 8) * 2 + 16 * (LBN + 8) * 2 + 4 * 16 * 4 + kDecodePages * 4 + 1024;
+  const long long slots = (long long)latent_sm_count() * max(1, min(8, (227 * 1024) / smem));
+  int best = 1;
+  long long best_cost = -1;
+  for (int splits = 1; splits <= most; ++splits) {
+    const long long rounds = (rows * splits + slots - 1) / slots;
+    const long long cost = 8 * rounds * ((tiles + splits - 1) / splits + 3) + splits;
+    if (best_cost < 0 || cost < best_cost) {
+      best = splits;
+      best_cost = cost;
+    }
+  }
+  return best;
 }
 
 // q_full [n_tokens, heads, rank + rot] and out [n_tokens, heads, rank] bfloat16; cache [pages, page_size, rank + rot];

@@ -225,15 +225,18 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, int q_col
 //   key pool        =        rotate(w_k[i] * k[n, i] / sqrt(mean(k[n]^2) + eps))    likewise over n_kv d entries
 //   value pool      =        v[n]
 // with t(p) = 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) at position p (temp_every <= 0: 1).  Columns, pools, slots and
-// rotation as qkv_prepare_kernel's; null weights: no norm.  `wide`: no rotation, head sizes and columns are multiples of eight
-// and every array lies on 16-byte boundaries: pieces of eight numbers.
+// rotation as qkv_prepare_kernel's; null weights: no norm.
+__device__ __forceinline__ float query_temperature(int position, float coef, double every) {
+  return every > 0.0 ? 1.f + coef * logf((float)(floor((double)(position + 1) / every) + 1.0)) : 1.f;
+}
+
 template <typename T>
 __global__ void qkv_prepare_rows_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col, int v_col, int n_q, int n_kv,
                                         int d, int dv, const int* __restrict__ slots, const float* __restrict__ q_weight,
                                         const float* __restrict__ k_weight, float eps, const float2* __restrict__ cos_sin,
                                         int rotary_dim, int interleaved, const int* __restrict__ positions, float temp_coef,
                                         double temp_every, T* __restrict__ k_pool, T* __restrict__ v_pool, int page_size,
-                                        T* __restrict__ q_out, int wide) {
+                                        T* __restrict__ q_out) {
   grid_dependency_wait();
   grid_dependency_launch();
   __shared__ float scratch[32];
@@ -242,60 +245,14 @@ __global__ void qkv_prepare_rows_kernel(const T* __restrict__ proj, int ld, int 
   const T *q = row + q_col, *k = row + k_col, *v = row + v_col;
   const int q_size = n_q * d, k_size = n_kv * d, v_size = n_kv * dv;
   float q_sq = 0.f, k_sq = 0.f;
-  if (wide) {
-    if (q_weight)
-      for (int i = threadIdx.x * 8; i < q_size; i += blockDim.x * 8) {
-        const Vec8 x = load8(q + i);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) q_sq += x.v[e] * x.v[e];
-      }
-    if (k_weight)
-      for (int i = threadIdx.x * 8; i < k_size; i += blockDim.x * 8) {
-        const Vec8 x = load8(k + i);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) k_sq += x.v[e] * x.v[e];
-      }
-  } else {
-    if (q_weight)
-      for (int i = threadIdx.x; i < q_size; i += blockDim.x) q_sq += to_float(q[i]) * to_float(q[i]);
-    if (k_weight)
-      for (int i = threadIdx.x; i < k_size; i += blockDim.x) k_sq += to_float(k[i]) * to_float(k[i]);
-  }
+  for (int i = threadIdx.x; i < q_size; i += blockDim.x) q_sq += to_float(q[i]) * to_float(q[i]);
+  for (int i = threadIdx.x; i < k_size; i += blockDim.x) k_sq += to_float(k[i]) * to_float(k[i]);
   float q_factor = 1.f, k_factor = 1.f;
   if (q_weight) q_factor = 1.0f / sqrtf(block_sum(q_sq, scratch) / (float)q_size + eps);
   if (k_weight) k_factor = 1.0f / sqrtf(block_sum(k_sq, scratch) / (float)k_size + eps);
-  if (temp_every > 0.0) q_factor *= 1.f + temp_coef * logf((float)(floor((double)(positions[n] + 1) / temp_every) + 1.0));
+  if (temp_every > 0.0) q_factor *= query_temperature(positions[n], temp_coef, temp_every);
   const int slot = slots[n];
   const int page = slot < 0 ? 0 : slot / page_size, offset = slot < 0 ? 0 : slot % page_size;
-  if (wide) {
-    for (int i = threadIdx.x * 8; i < q_size; i += blockDim.x * 8) {
-      Vec8 x = load8(q + i);
-      if (q_weight) {
-        const Vec8 w = load8(q_weight + i);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x.v[e] *= w.v[e];
-      }
-#pragma unroll
-      for (int e = 0; e < 8; ++e) x.v[e] *= q_factor;
-      store8(q_out + n * q_size + i, x);
-    }
-    if (slot < 0) return;
-    for (int i = threadIdx.x * 8; i < k_size; i += blockDim.x * 8) {
-      Vec8 x = load8(k + i);
-      if (k_weight) {
-        const Vec8 w = load8(k_weight + i);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x.v[e] *= w.v[e] * k_factor;
-      }
-      const int g = i / d;
-      store8(k_pool + (((size_t)page * n_kv + g) * page_size + offset) * d + (i - g * d), x);
-    }
-    for (int i = threadIdx.x * 8; i < v_size; i += blockDim.x * 8) {
-      const int g = i / dv;
-      store8(v_pool + (((size_t)page * n_kv + g) * page_size + offset) * dv + (i - g * dv), load8(v + i));
-    }
-    return;
-  }
   const int half = rotary_dim >> 1;
   const float2* table = cos_sin ? cos_sin + n * half : nullptr;
   auto value = [&](const T* src, const float* weight, float factor, int i) {      // entry i of a normed row, rotated
@@ -320,6 +277,105 @@ __global__ void qkv_prepare_rows_kernel(const T* __restrict__ proj, int ld, int 
   for (int i = threadIdx.x; i < v_size; i += blockDim.x) {
     const int g = i / dv;
     v_pool[(((size_t)page * n_kv + g) * page_size + offset) * dv + (i - g * dv)] = v[i];
+  }
+}
+
+// The same without rotation where head sizes and columns are multiples of eight and every array lies on 16-byte boundaries: a
+// thread holds up to PIECES pieces of eight numbers of queries, keys and values in registers, so a row is read once, and both
+// sums of squares meet in one exchange.  A block takes every gridDim.x-th token; a piece's place in its head and (where PIECES
+// is one) its norm weights are found once, the weights while the kernel before ends.  What a token needs once (its page, its
+// temperature) is one thread's work.
+template <typename T, int PIECES>
+__global__ void __launch_bounds__(512, PIECES == 1 ? 3 : 2)
+qkv_prepare_rows_vec_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col, int v_col, int n_q, int n_kv, int d, int dv,
+                            const int* __restrict__ slots, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
+                            float eps, const int* __restrict__ positions, float temp_coef, double temp_every, T* __restrict__ k_pool,
+                            T* __restrict__ v_pool, int page_size, T* __restrict__ q_out, int n_tokens) {
+  constexpr bool KEPT = PIECES == 1;
+  enum : int { QUERY = 0, KEY = 1, VALUE = 2, NONE = 3 };
+  const int q_size = n_q * d, k_size = n_kv * d, all = q_size + k_size + n_kv * dv;
+  Vec8 w[PIECES], x[PIECES];
+  int kind[PIECES], column[PIECES], target[PIECES];      // what a piece is, where it lies in proj's row, and in q_out's or its page
+  auto weight_of = [&](int i) {
+    const float* source = kind[i] == QUERY ? q_weight : kind[i] == KEY ? k_weight : nullptr;
+    if (source) {
+      w[i] = load8(source + (kind[i] == QUERY ? column[i] - q_col : column[i] - k_col));
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w[i].v[e] = 1.f;
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < PIECES; ++i) {
+    int at = (i * (int)blockDim.x + (int)threadIdx.x) * 8;
+    kind[i] = at >= all ? NONE : at < q_size ? QUERY : at < q_size + k_size ? KEY : VALUE;
+    column[i] = target[i] = 0;
+    if (kind[i] == QUERY) {
+      column[i] = q_col + at;
+      target[i] = at;
+    } else if (kind[i] != NONE) {
+      at -= kind[i] == KEY ? q_size : q_size + k_size;
+      const int size = kind[i] == KEY ? d : dv, g = at / size;
+      column[i] = (kind[i] == KEY ? k_col : v_col) + at;
+      target[i] = g * page_size * size + (at - g * size);
+    }
+    if (KEPT) weight_of(i);
+  }
+  grid_dependency_wait();
+  grid_dependency_launch();
+  __shared__ float2 sums[2][32];
+  __shared__ float temperature[2];
+  __shared__ long long first_row[2];                        // of the token's slot: page * n_kv * page_size + offset; -1: not stored
+  const bool single = threadIdx.x == blockDim.x - 1;
+  int slot = 0, position = 0;
+  if (single && (int)blockIdx.x < n_tokens) {
+    slot = slots[blockIdx.x];
+    position = temp_every > 0.0 ? positions[blockIdx.x] : 0;
+  }
+  for (int n = blockIdx.x, turn = 0; n < n_tokens; n += gridDim.x, turn ^= 1) {
+    if (single) {
+      const int page = slot < 0 ? 0 : slot / page_size;
+      first_row[turn] = slot < 0 ? -1 : (long long)page * n_kv * page_size + (slot - page * page_size);
+      temperature[turn] = query_temperature(position, temp_coef, temp_every);
+      if (n + (int)gridDim.x < n_tokens) {
+        slot = slots[n + gridDim.x];
+        position = temp_every > 0.0 ? positions[n + gridDim.x] : 0;
+      }
+    }
+    const T* row = proj + (size_t)n * ld;
+    float2 sq = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+      if (kind[i] == NONE) continue;
+      x[i] = load8(row + column[i]);
+      float sum = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sum += x[i].v[e] * x[i].v[e];
+      if (kind[i] == QUERY) sq.x += sum;
+      if (kind[i] == KEY) sq.y += sum;
+    }
+    sq.x = warp_sum(sq.x);
+    sq.y = warp_sum(sq.y);
+    if ((threadIdx.x & 31) == 0) sums[turn][threadIdx.x >> 5] = sq;
+    __syncthreads();                                        // (the next token's sums go to the other half)
+    sq = make_float2(0.f, 0.f);
+    for (int i = 0; i < (int)(blockDim.x >> 5); ++i) {
+      sq.x += sums[turn][i].x;
+      sq.y += sums[turn][i].y;
+    }
+    const long long first = first_row[turn];
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+      if (kind[i] == NONE) continue;
+      if (!KEPT) weight_of(i);
+      float factor = 1.f;
+      if (kind[i] == QUERY) factor = (q_weight ? 1.0f / sqrtf(sq.x / (float)q_size + eps) : 1.f) * temperature[turn];
+      if (kind[i] == KEY && k_weight) factor = 1.0f / sqrtf(sq.y / (float)k_size + eps);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[i].v[e] *= w[i].v[e] * factor;
+      if (kind[i] == QUERY) store8(q_out + (size_t)n * q_size + target[i], x[i]);
+      else if (first >= 0) store8(kind[i] == KEY ? k_pool + first * d + target[i] : v_pool + first * dv + target[i], x[i]);
+    }
   }
 }
 
@@ -389,6 +445,23 @@ MS_EXPORT int ms_qkv_prepare(const void* proj, int dtype, int ld, int q_col, int
   return 0;
 }
 
+// Thread blocks of `threads` threads of this kernel that the GPU holds at once (kept per kernel and block size).
+template <auto Kernel>
+static int resident_blocks(int threads) {
+  static int known[33] = {};
+  int& count = known[threads / 32];
+  if (count == 0) {
+    int device = 0, sms = 0, per_sm = 0;
+    if (cudaGetDevice(&device) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) != cudaSuccess ||
+        cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, Kernel, threads, 0) != cudaSuccess || sms * per_sm <= 0) {
+      cudaGetLastError();
+      return 148;
+    }
+    count = sms * per_sm;
+  }
+  return count;
+}
+
 // proj [n_tokens, ld]; norm weights float32 [n_q d] and [n_kv d] (null: no norm); positions int32 [n_tokens] (read where temp_every > 0).
 MS_EXPORT int ms_qkv_prepare_rows(const void* proj, int dtype, int ld, int q_col, int k_col, int v_col, int n_q, int n_kv, int d,
                                   int dv, const int* slots, const float* q_weight, const float* k_weight, float eps,
@@ -403,11 +476,27 @@ MS_EXPORT int ms_qkv_prepare_rows(const void* proj, int dtype, int ld, int q_col
   auto aligned = [](const void* p) { return reinterpret_cast<size_t>(p) % 16 == 0; };
   const int wide = rotary_dim == 0 && d % 8 == 0 && dv % 8 == 0 && ld % 8 == 0 && q_col % 8 == 0 && k_col % 8 == 0 && v_col % 8 == 0 &&
                    aligned(proj) && aligned(q_out) && aligned(k_pool) && aligned(v_pool) && aligned(q_weight) && aligned(k_weight);
+  const int pieces = ((n_q + n_kv) * d + n_kv * dv) / 8;
+  if (wide && pieces <= 4 * 512) {
+    const int each = pieces <= 512 ? 1 : pieces <= 1024 ? 2 : 4;
+    const int threads = ((pieces + each - 1) / each + 31) / 32 * 32;
+#define MS_PREPARE_ROWS(P)                                                                                                      \
+  MS_EG_DISPATCH(dtype, {                                                                                                       \
+    const int slots_on_gpu = resident_blocks<qkv_prepare_rows_vec_kernel<T, P>>(threads);                                        \
+    ms::launch(qkv_prepare_rows_vec_kernel<T, P>, n_tokens < slots_on_gpu ? n_tokens : slots_on_gpu, threads, 0, stream,        \
+               (const T*)proj, ld, q_col, k_col, v_col, n_q, n_kv, d, dv, slots, q_weight, k_weight, eps, positions, temp_coef, \
+               (double)temp_every, (T*)k_pool, (T*)v_pool, page_size, (T*)q_out, n_tokens);                                     \
+  })
+    if (each == 1) { MS_PREPARE_ROWS(1); } else if (each == 2) { MS_PREPARE_ROWS(2); } else { MS_PREPARE_ROWS(4); }
+#undef MS_PREPARE_ROWS
+    MS_CHECK_LAUNCH("qkv_prepare_rows");
+    return 0;
+  }
   const int threads = n_q * d >= 2048 ? 256 : 128;
   MS_EG_DISPATCH(dtype, (ms::launch(qkv_prepare_rows_kernel<T>, n_tokens, threads, 0, stream, (const T*)proj, ld, q_col, k_col, v_col,
                                     n_q, n_kv, d, dv, slots, q_weight, k_weight, eps, (const float2*)(rotary_dim ? cos_sin : nullptr),
                                     rotary_dim, interleaved, positions, temp_coef, (double)temp_every, (T*)k_pool, (T*)v_pool,
-                                    page_size, (T*)q_out, wide)));
+                                    page_size, (T*)q_out)));
   MS_CHECK_LAUNCH("qkv_prepare_rows");
   return 0;
 }
@@ -520,7 +609,7 @@ __global__ void sigmoid_gate_mul_vec_kernel(const T* __restrict__ x, const T* __
   grid_dependency_launch();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= pieces) return;
-  const size_t n = i / per_row;
+  const size_t n = pieces <= 0xffffffffu ? (unsigned)i / (unsigned)per_row : i / per_row;      // 32-bit division where it is enough
   const Vec8 g = load8(gate + n * gate_ld + gate_col + (i - n * per_row) * 8);
   Vec8 v = load8(x + i * 8);
 #pragma unroll

@@ -56,13 +56,25 @@ __global__ void add_layernorm_kernel(float* __restrict__ residual, const T* __re
 }
 
 // The same with sixteen-byte loads and stores: each thread keeps up to CHUNKS groups of eight elements in registers, so every
-// row is read once.  Requires hidden % 8 == 0 and hidden <= 8 * blockDim.x * CHUNKS.
-template <typename T, int CHUNKS>
+// row is read once.  Requires hidden % 8 == 0 and hidden <= 8 * blockDim.x * CHUNKS.  EARLY (one group a thread, launches of few
+// rows): weights and biases, which are no kernel's output, are fetched while the kernel before ends; in launches of many rows
+// the registers that hold them cost more than their wait.
+template <typename T, int CHUNKS, bool EARLY>
 __global__ void add_layernorm_vec_kernel(float* __restrict__ residual, const T* __restrict__ delta, const T* __restrict__ delta2,
                                          const float* __restrict__ vector, const void* __restrict__ weight,
                                          const void* __restrict__ bias, const void* __restrict__ weight2,
                                          const void* __restrict__ bias2, int weight_dtype, float eps, const int* __restrict__ rows,
                                          T* __restrict__ out, T* __restrict__ out2, int hidden) {
+  static_assert(!EARLY || CHUNKS == 1, "one group a thread");
+  Vec8 w, b, w2, b2;
+  if (EARLY && (int)threadIdx.x * 8 < hidden) {
+    w = load8_any(weight, weight_dtype, threadIdx.x * 8);
+    b = load8_any(bias, weight_dtype, threadIdx.x * 8);
+    if (out2) {
+      w2 = load8_any(weight2, weight_dtype, threadIdx.x * 8);
+      b2 = load8_any(bias2, weight_dtype, threadIdx.x * 8);
+    }
+  }
   grid_dependency_wait();
   grid_dependency_launch();
   __shared__ float scratch[32];
@@ -117,13 +129,19 @@ __global__ void add_layernorm_vec_kernel(float* __restrict__ residual, const T* 
   for (int i = 0; i < CHUNKS; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * 8;
     if (c < hidden) {
-      const Vec8 w = load8_any(weight, weight_dtype, c), b = load8_any(bias, weight_dtype, c);
+      if (!EARLY) {
+        w = load8_any(weight, weight_dtype, c);
+        b = load8_any(bias, weight_dtype, c);
+      }
       Vec8 y;
 #pragma unroll
       for (int e = 0; e < 8; ++e) y.v[e] = w.v[e] * (x[i].v[e] * inv) + b.v[e];
       store8(out + k * hidden + c, y);
       if (out2) {
-        const Vec8 w2 = load8_any(weight2, weight_dtype, c), b2 = load8_any(bias2, weight_dtype, c);
+        if (!EARLY) {
+          w2 = load8_any(weight2, weight_dtype, c);
+          b2 = load8_any(bias2, weight_dtype, c);
+        }
 #pragma unroll
         for (int e = 0; e < 8; ++e) y.v[e] = w2.v[e] * (x[i].v[e] * inv) + b2.v[e];
         store8(out2 + k * hidden + c, y);
@@ -186,11 +204,12 @@ MS_EXPORT int ms_add_layernorm(float* residual, const void* delta, const void* d
     const int groups = hidden / 8;
     const int threads = groups >= 256 ? 256 : ((groups + 31) / 32) * 32;
     const int chunks = (groups + threads - 1) / threads;
-#define MS_LN_VEC(C)                                                                                                             \
-  MS_LN_DISPATCH(dtype, (ms::launch(add_layernorm_vec_kernel<T, C>, n_out, threads, 0, stream, residual, (const T*)delta,        \
+#define MS_LN_VEC(C, E)                                                                                                             \
+  MS_LN_DISPATCH(dtype, (ms::launch(add_layernorm_vec_kernel<T, C, E>, n_out, threads, 0, stream, residual, (const T*)delta,        \
                                     (const T*)delta2, vector, weight, bias, weight2, bias2, weight_dtype, eps, rows, (T*)out,    \
                                     (T*)out2, hidden)))
-    if (chunks == 1) { MS_LN_VEC(1); } else if (chunks == 2) { MS_LN_VEC(2); } else { MS_LN_VEC(4); }
+    if (chunks == 1 && n_out <= 256) { MS_LN_VEC(1, true); } else if (chunks == 1) { MS_LN_VEC(1, false); }
+    else if (chunks == 2) { MS_LN_VEC(2, false); } else { MS_LN_VEC(4, false); }
 #undef MS_LN_VEC
     MS_CHECK_LAUNCH("add_layernorm");
     return 0;

@@ -95,7 +95,8 @@ def test_stream_to_columns_kernel(dtype, hidden, ld, col):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("n_q,n_kv,d,dv,rotary,interleaved", [(4, 2, 16, 24, 0, False), (3, 3, 7, 9, 0, False), (8, 1, 64, 64, 0, False),
-                                                              (6, 2, 20, 12, 8, True), (2, 1, 12, 8, 12, False), (32, 8, 128, 128, 0, False)])
+                                                              (6, 2, 20, 12, 8, True), (2, 1, 12, 8, 12, False), (32, 8, 128, 128, 0, False),
+                                                              (64, 16, 64, 64, 0, False), (64, 16, 128, 64, 0, False), (128, 16, 128, 64, 0, False)])
 @pytest.mark.parametrize("temperature", [None, (0.4, 3.0), (-0.2, 1.0)])
 def test_prepare_with_norms_over_the_whole_row(dtype, n_q, n_kv, d, dv, rotary, interleaved, temperature):
     from miniserve_b200 import kernels
@@ -121,6 +122,28 @@ def test_prepare_with_norms_over_the_whole_row(dtype, n_q, n_kv, d, dv, rotary, 
                                    temperature=temperature)
         for got, expected in zip((q, k_pool, v_pool), want):
             assert close(got, expected, dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_prepare_with_norms_over_the_whole_row_of_many_tokens(dtype):
+    """More tokens than blocks: every block takes several, fetching the next row while it works on one."""
+    from miniserve_b200 import kernels
+
+    n, n_q, n_kv, d, dv, page = 2500, 4, 2, 16, 24, 16
+    proj = rand((n, n_q * d + n_kv * (d + dv)), dtype, 1, 2.0)
+    qw, kw = 1 + rand((n_q * d,), torch.float32, 2, 0.3), 1 + rand((n_kv * d,), torch.float32, 3, 0.3)
+    slots = torch.randperm(n, generator=torch.Generator().manual_seed(4)).to(torch.int32)
+    slots[::97] = -1
+    k_pool, v_pool = torch.zeros((160, n_kv, page, d), dtype=dtype).cuda(), torch.zeros((160, n_kv, page, dv), dtype=dtype).cuda()
+    q = torch.empty((n, n_q, d), dtype=dtype).cuda()
+    want = [torch.zeros(t.shape, dtype=torch.float64) for t in (q, k_pool, v_pool)]
+    positions = torch.arange(n, dtype=torch.int32)
+    kernels.qkv_prepare_rows(proj, 0, 64, 96, n_q, n_kv, d, dv, slots.cuda(), qw, kw, 1e-5, None, 0, k_pool, v_pool, q,
+                             positions=positions.cuda(), temperature=(0.3, 100.0))
+    plain_ops.qkv_prepare_rows(cpu(proj), 0, 64, 96, n_q, n_kv, d, dv, slots, cpu(qw), cpu(kw), 1e-5, None, 0, want[1], want[2], want[0],
+                               positions=positions, temperature=(0.3, 100.0))
+    for got, expected in zip((q, k_pool, v_pool), want):
+        assert close(got, expected, dtype)
 
 
 def attention_case(dtype, n_q, n_kv, d, dv, page, queries, contexts, seed=0):
