@@ -293,8 +293,9 @@ class CacheManager:
             tables = [table + new for table, new in zip(entry.tables, new_pages)]
             slots = []
             positions = numpy.arange(entry.length, end, dtype=numpy.int64)
+            first_page = entry.length // self.page_size            # (only the pages that the new tokens fall into are looked at)
             for table in tables:
-                pages = numpy.asarray(table, dtype=numpy.int64)[positions // self.page_size]
+                pages = numpy.asarray(table[first_page:], dtype=numpy.int64)[positions // self.page_size - first_page]
                 if (pages == RELEASED).any():
                     raise RuntimeError("a new token falls into a page that was given back")
                 slots.append(pages * self.page_size + positions % self.page_size)
@@ -322,12 +323,12 @@ class CacheManager:
                 # the next query sits at position `length`; it sees keys from length - window + 1 on (or from its chunk's start)
                 first_needed = need.first_needed(entry.length)
                 table = entry.tables[group]
-                for index in range(len(table)):
-                    if (index + 1) * self.page_size > first_needed:
-                        break
-                    if table[index] != RELEASED:
-                        self.allocators[group].release(table[index])
-                        table[index] = RELEASED
+                # the pages wholly before it; those given back at earlier commits are the table's first ones
+                index = min(first_needed // self.page_size, len(table)) - 1
+                while index >= 0 and table[index] != RELEASED:
+                    self.allocators[group].release(table[index])
+                    table[index] = RELEASED
+                    index -= 1
 
     def abort(self, reservation: StepReservation) -> None:
         self._close(reservation)
