@@ -955,7 +955,7 @@ class BafavikConfig:
 
 
 def _window_or_none(data: Mapping[str, Any], where: str) -> Any:
-    """``mask.size`` of a mixer whose tokens see themselves and the ``size - 1`` tokens before them (no ``mask``: every token)."""
+    """``mask.size``: how many of the latest keys, its own included, a query sees (no ``mask``: all)."""
     if data.get("mask") is None:
         return None
     return _integer(_section(data, "mask", where), "size")
