@@ -1093,3 +1093,215 @@ class VenaraxConfig:
                   for layer in self.layers]
         loop = None if self.loop is None else dict(start=self.loop[0], stop=self.loop[1], times=self.loop[2])
         return dict(architecture=self.architecture, vocab=self.vocab, width=self.width, norm=dict(eps=self.eps), loop=loop, layers=layers)
+
+
+# --------------------------------------------------------------------------- Parunex
+
+
+@dataclass(frozen=True)
+class WavelengthRotationConfig:
+    """A rotary position encoding over ``dims`` entries (0: none) whose frequencies may be scaled by wavelength: ``scaling`` is None
+    or the constants (factor, low, high, original)."""
+
+    base: float
+    dims: int
+    scaling: Any = None
+
+    SCALING = ("factor", "low", "high", "original")
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], where: str) -> "WavelengthRotationConfig":
+        scaling = None
+        if data.get("scaling") is not None:
+            section = _section(data, "scaling", where)
+            scaling = tuple(_positive(section, key, where + "scaling.") for key in cls.SCALING)
+        config = cls(base=_positive(data, "base", where), dims=_count(data, "dims", 0), scaling=scaling)
+        if config.dims % 2:
+            raise ValueError(f"{where}dims {config.dims} is odd; the rotation turns pairs of entries")
+        return config
+
+    def scaling_dict(self):
+        return None if self.scaling is None else dict(zip(self.SCALING, self.scaling))
+
+    def to_dict(self) -> dict[str, Any]:
+        out: dict[str, Any] = dict(base=self.base, dims=self.dims)
+        if self.scaling is not None:
+            out["scaling"] = self.scaling_dict()
+        return out
+
+
+@dataclass(frozen=True)
+class CappedAttentionConfig:
+    """Grouped-query attention with biases on queries, keys and values, a rotation of the first ``rot.dims`` entries, scores with a
+    soft cap (``softcap``, or None), a learned sink and a gate per head.  ``v_mix``: the layer takes part in the mixing of values
+    along the depth (the first such layer gives its values to the others)."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: WavelengthRotationConfig
+    softcap: Any = None
+    v_mix: bool = False
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], where: str) -> "CappedAttentionConfig":
+        config = cls(heads=_integer(data, "heads"), kv_heads=_integer(data, "kv_heads"), dim=_integer(data, "dim"),
+                     vdim=_integer(data, "vdim"), scale=_positive(data, "scale", where),
+                     rot=WavelengthRotationConfig.from_dict(_section(data, "rot", where), where + "rot."),
+                     softcap=None if data.get("softcap") is None else _positive(data, "softcap", where),
+                     v_mix=_boolean(data, "v_mix"))
+        if config.heads % config.kv_heads:
+            raise ValueError(f"{where}heads {config.heads} is not a multiple of kv_heads {config.kv_heads}")
+        if config.rot.dims > config.dim:
+            raise ValueError(f"{where}rot.dims {config.rot.dims} exceeds the head size dim {config.dim}")
+        return config
+
+    def to_dict(self) -> dict[str, Any]:
+        out: dict[str, Any] = dict(heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, scale=self.scale,
+                                   rot=self.rot.to_dict(), v_mix=self.v_mix)
+        if self.softcap is not None:
+            out["softcap"] = self.softcap
+        return out
+
+
+@dataclass(frozen=True)
+class GatedLinearAttentionConfig:
+    """Gated linear attention: ``heads`` heads with queries and keys of ``dim`` and values of ``vdim`` entries, a decay per key channel
+    to the power ``1 / tau``.  ``rank``, the inner size of the decay's two-step projection, comes from a checkpoint's tensor shapes
+    where ``config.json`` does not give it."""
+
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: Any = None
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], where: str) -> "GatedLinearAttentionConfig":
+        return cls(heads=_integer(data, "heads"), dim=_integer(data, "dim"), vdim=_integer(data, "vdim"), tau=_positive(data, "tau", where),
+                   rank=_integer(data, "rank") if "rank" in data else None)
+
+    def to_dict(self) -> dict[str, Any]:
+        out: dict[str, Any] = dict(heads=self.heads, dim=self.dim, vdim=self.vdim, tau=self.tau)
+        if self.rank is not None:
+            out["rank"] = self.rank
+        return out
+
+
+@dataclass(frozen=True)
+class ParunexFeedForwardConfig:
+    """``kind`` "dense": a gated feed-forward of inner size ``ff``.  ``kind`` "moe": ``experts`` gated experts of inner size ``ff``, of
+    which a token uses ``top`` among those of the ``group_keep`` best of ``group_count`` groups; ``scale`` multiplies the weights."""
+
+    kind: str
+    ff: int
+    experts: int = 0
+    top: int = 0
+    scale: float = 1.0
+    group_count: int = 1
+    group_keep: int = 1
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], where: str) -> "ParunexFeedForwardConfig":
+        kind = data.get("kind")
+        if kind == "dense":
+            return cls(kind="dense", ff=_integer(data, "ff"))
+        if kind != "moe":
+            raise UnsupportedModelError(f"UNSUPPORTED_MODEL_CONFIGURATION: {where}kind {kind!r} is not implemented (dense, moe)")
+        router = _section(data, "router", where)
+        count, keep = 1, 1
+        if router.get("groups") is not None:
+            groups = _section(router, "groups", where + "router.")
+            count, keep = _integer(groups, "count"), _integer(groups, "keep")
+        scale = _number(router, "scale")
+        if not math.isfinite(scale):
+            raise ValueError(f"{where}router.scale must be finite, got {scale}")
+        config = cls(kind="moe", ff=_integer(_section(data, "expert", where), "ff"), experts=_integer(router, "experts"),
+                     top=_integer(router, "top"), scale=scale, group_count=count, group_keep=keep)
+        if config.experts % count or keep > count:
+            raise ValueError(f"{where}router.groups: {config.experts} experts in {count} groups, {keep} kept")
+        if config.top > keep * (config.experts // count):
+            raise ValueError(f"{where}router.top {config.top} exceeds the {keep} kept groups of {config.experts // count}")
+        return config
+
+    def to_dict(self) -> dict[str, Any]:
+        if self.kind == "dense":
+            return dict(kind="dense", ff=self.ff)
+        router: dict[str, Any] = dict(experts=self.experts, top=self.top, scale=self.scale,
+                                      groups=dict(count=self.group_count, keep=self.group_keep))
+        return dict(kind="moe", expert=dict(ff=self.ff), router=router)
+
+
+@dataclass(frozen=True)
+class ParunexLayerConfig:
+    type: str       # "attention" or "gla"
+    mixer: Any
+    mlp: Any        # ParunexFeedForwardConfig or None
+
+
+@dataclass(frozen=True)
+class ParunexConfig:
+    """The Parunex decoder: ``config.json`` holds ``architecture``, ``vocab``, ``width``, ``embedding.scale``, ``norm.eps`` and ``layers``, a
+    list whose entries give each layer's mixer ``type`` (``attention`` or ``gla``), the mixer's sizes and constants (``mixer``) and its
+    feed-forward (``mlp``, or null).  Every size and constant is read."""
+
+    vocab: int
+    width: int
+    embedding_scale: float
+    eps: float
+    layers: tuple
+    architecture: str = "Parunex"
+
+    MIXERS = {"attention": CappedAttentionConfig.from_dict, "gla": GatedLinearAttentionConfig.from_dict}
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any]) -> "ParunexConfig":
+        if data.get("architecture") != "Parunex":
+            raise UnsupportedModelError(f"UNSUPPORTED_MODEL_CONFIGURATION: expected architecture 'Parunex', got {data.get('architecture')!r}")
+        raw_layers = data.get("layers")
+        if not isinstance(raw_layers, (list, tuple)) or not raw_layers:
+            raise ValueError("layers must be a non-empty list in the model config")
+        layers, giver = [], None
+        for index, raw in enumerate(raw_layers):
+            where = f"layers[{index}]."
+            if not isinstance(raw, Mapping):
+                raise ValueError(f"layers[{index}] must be an object")
+            kind = raw.get("type")
+            if kind not in cls.MIXERS:
+                raise UnsupportedModelError(f"UNSUPPORTED_MODEL_CONFIGURATION: {where}type {kind!r} is not implemented "
+                                            f"({', '.join(cls.MIXERS)})")
+            mixer = cls.MIXERS[kind](_section(raw, "mixer", where), where + "mixer.")
+            if kind == "attention" and mixer.v_mix:
+                giver = mixer if giver is None else giver
+                if giver.kv_heads * giver.vdim != mixer.kv_heads * mixer.vdim:
+                    raise ValueError(f"{where}mixer.v_mix: {mixer.kv_heads} value heads of {mixer.vdim} cannot be mixed with the first "
+                                     f"such layer's {giver.kv_heads} of {giver.vdim}")
+            mlp = None if raw.get("mlp") is None else ParunexFeedForwardConfig.from_dict(_section(raw, "mlp", where), where + "mlp.")
+            layers.append(ParunexLayerConfig(kind, mixer, mlp))
+        scale = _number(_section(data, "embedding", ""), "scale")
+        if not math.isfinite(scale):
+            raise ValueError(f"embedding.scale must be finite, got {scale}")
+        return cls(vocab=_integer(data, "vocab"), width=_integer(data, "width"), embedding_scale=scale,
+                   eps=_positive(_section(data, "norm", ""), "eps", "norm."), layers=tuple(layers))
+
+    def with_stored_shapes(self, shapes: Mapping[str, tuple]) -> "ParunexConfig":
+        """The configuration with the sizes that only a checkpoint's tensor shapes give: the inner sizes of the decays' two-step
+        projections (the rows of ``l<i>.mix.a1``)."""
+        from dataclasses import replace
+
+        layers = []
+        for index, layer in enumerate(self.layers):
+            stored = shapes.get(f"l{index}.mix.a1")
+            if layer.type == "gla" and layer.mixer.rank is None and stored is not None and len(stored) == 2:
+                layer = replace(layer, mixer=replace(layer.mixer, rank=int(stored[0])))
+            layers.append(layer)
+        return replace(self, layers=tuple(layers))
+
+    def to_dict(self) -> dict[str, Any]:
+        """The ``config.json`` content that reads back as this configuration."""
+        layers = [dict(type=layer.type, mixer=layer.mixer.to_dict(), mlp=None if layer.mlp is None else layer.mlp.to_dict())
+                  for layer in self.layers]
+        return dict(architecture=self.architecture, vocab=self.vocab, width=self.width, embedding=dict(scale=self.embedding_scale),
+                    norm=dict(eps=self.eps), layers=layers)

@@ -30,7 +30,7 @@ attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
                      int n_kv, float scale_log2, int window, __nv_bfloat16* __restrict__ out,
                      float* __restrict__ part_o, float* __restrict__ part_lse, int num_splits, int sink,
                      const float* __restrict__ sink_scores,
-                     const __nv_bfloat16* __restrict__ gate, int gate_ld) {
+                     const __nv_bfloat16* __restrict__ gate, int gate_ld, float cap_log2) {
   // The kernel before this one on the stream wrote the queries and the keys and values of this step's
   // tokens.  What the batch looks like (set up before the step's first kernel) and the keys and values of
   // earlier steps do not depend on it, so the first tiles of old keys are requested before the wait below.
@@ -230,6 +230,15 @@ attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
       }
     }
 
+    if (cap_log2 > 0.f) {                  // scores under a soft cap: from here on their tanh, scaled by the cap
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int n = 0; n < BN / 8; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc_s[mt][n][e] = capped_score(acc_s[mt][n][e], cap_log2);
+    }
+
     // ---- mask and online softmax (scores are scaled inside the exponent)
     const bool full = (key0 + BN - 1 <= first_pos + t_lo) && (window <= 0 || key0 >= first_pos + t_hi - window + 1);
 #pragma unroll
@@ -370,7 +379,7 @@ int launch_attention_mma(const void* q, const void* k_pool, const void* v_pool, 
                          int table_stride, const int* query_start, const int* context_lens, int page_size, int n_q,
                          int n_kv, float scale, int window, void* out, float* part_o, float* part_lse, int num_splits,
                          int n_requests, int max_query_len, int n_tokens, int sink, const float* sink_scores, const void* gate,
-                         int gate_ld, int first_token, cudaStream_t stream) {
+                         int gate_ld, int first_token, float softcap, cudaStream_t stream) {
   constexpr int BM = 16 * MT * W;
   const size_t smem = (size_t)(BM + 2 * STAGES * BN) * D * sizeof(__nv_bfloat16) + STAGES * BN * sizeof(long long);
   auto kernel = attention_mma_kernel<D, W, BN, MT, STAGES>;
@@ -385,11 +394,12 @@ int launch_attention_mma(const void* q, const void* k_pool, const void* v_pool, 
   MS_REQUIRE(tiles <= 2147483647LL && (long long)n_requests * num_splits <= 65535 && n_kv <= 65535,
              "attention: grid %lld x %d x %lld exceeds the launch limits", tiles, n_kv, (long long)n_requests * num_splits);
   dim3 grid((unsigned)tiles, n_kv, n_requests * num_splits);
-  const float scale_log2 = scale * 1.4426950408889634f;
+  const float scale_log2 = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f;
+  const float cap_log2 = softcap > 0.f ? 2.f * scale / softcap * 1.4426950408889634f : 0.f;
   ms::launch(kernel, grid, W * 32, smem, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool,
                                          (const __nv_bfloat16*)v_pool, block_tables, table_stride, query_start,
                                          context_lens, page_size, n_q, n_kv, scale_log2, window, (__nv_bfloat16*)out,
-                                         part_o, part_lse, num_splits, sink, sink_scores, (const __nv_bfloat16*)gate, gate_ld);
+                                         part_o, part_lse, num_splits, sink, sink_scores, (const __nv_bfloat16*)gate, gate_ld, cap_log2);
   MS_CHECK_LAUNCH("attention_mma");
   if (num_splits > 1) {
     // only the rows of this launch's requests (first_token .. n_tokens) hold partial results: the rows before them belong to
@@ -455,13 +465,14 @@ MS_EXPORT int ms_attention_mma_splits(int d, int n_requests, int n_kv, int n_q, 
 // exp(sink_scores[head]) where sink_scores (float32 [n_q]) is not null; gate (bfloat16 logits, gate[token * gate_ld +
 // head], or null): the head's output is multiplied by the sigmoid of its logit.  first_token: the first row that belongs to
 // these requests (rows before it are another launch's and are left alone).  num_splits > 1 needs part_o [n_tokens * n_q * num_splits * d] and part_lse
-// [n_tokens * n_q * num_splits] float32 scratch and is meant for steps of single tokens.
+// [n_tokens * n_q * num_splits] float32 scratch and is meant for steps of single tokens.  softcap c > 0: a scaled score s becomes
+// c tanh(s / c).
 MS_EXPORT int ms_paged_attention_mma(const void* q, const void* k_pool, const void* v_pool, const int* block_tables,
                                      int table_stride, const int* query_start, const int* context_lens,
                                      int page_size, int n_q, int n_kv, int d, float scale, int window, void* out,
                                      float* part_o, float* part_lse, int num_splits, int n_requests,
                                      int max_query_len, int n_tokens, int sink, const float* sink_scores, const void* gate,
-                                     int gate_ld, int first_token, cudaStream_t stream) {
+                                     int gate_ld, int first_token, float softcap, cudaStream_t stream) {
   if (n_tokens == 0 || n_requests == 0) return 0;
   MS_REQUIRE(first_token >= 0 && first_token < n_tokens, "attention: first row %d of %d", first_token, n_tokens);
   MS_REQUIRE(n_kv > 0 && n_q % n_kv == 0, "attention: %d query heads are not a multiple of %d key/value heads", n_q, n_kv);
@@ -474,7 +485,7 @@ MS_EXPORT int ms_paged_attention_mma(const void* q, const void* k_pool, const vo
 #define MS_ATTENTION_CASE(D, W, BN, MT, STAGES)                                                                       \
   return launch_attention_mma<D, W, BN, MT, STAGES>(q, k_pool, v_pool, block_tables, table_stride, query_start,       \
                                                     context_lens, page_size, n_q, n_kv, scale, window, out, part_o,  \
-                                                    part_lse, num_splits, n_requests, max_query_len, n_tokens, sink, sink_scores, gate, gate_ld, first_token, stream)
+                                                    part_lse, num_splits, n_requests, max_query_len, n_tokens, sink, sink_scores, gate, gate_ld, first_token, softcap, stream)
   if (d == 128) { if (small) { MS_ATTENTION_CASE(128, 1, 32, 1, 2); } else { MS_ATTENTION_CASE(128, 4, 64, 2, 2); } }
   if (d == 64) { if (small) { MS_ATTENTION_CASE(64, 1, 64, 1, 2); } else { MS_ATTENTION_CASE(64, 4, 64, 2, 2); } }
   if (d == 32) { if (small) { MS_ATTENTION_CASE(32, 1, 64, 1, 2); } else { MS_ATTENTION_CASE(32, 4, 64, 2, 2); } }
@@ -531,5 +542,5 @@ MS_EXPORT int ms_paged_attention_decode_static(const void* q, const void* k_pool
   // infinity when it had no keys), and a partial result is read only where that value is finite.
   return ms_paged_attention_mma(q, k_pool, v_pool, block_tables, table_stride, query_start, context_lens, page_size,
                                 n_q, n_kv, d, scale, window, out, part_o, part_lse, num_splits, n_requests, 1, n_tokens,
-                                0, nullptr, nullptr, 0, 0, stream);
+                                0, nullptr, nullptr, 0, 0, 0.f, stream);
 }

@@ -1,7 +1,7 @@
 // Paged grouped-query attention on the tensor cores for head sizes that attention_mma.cu is not built for: query and key
 // heads of d entries and value heads of dv entries, both any multiple of 16 up to 128 and not necessarily the same, with
-// the two options of the other kernels (a sink in the softmax's denominator, of score 0 or of a score per head; a gate per head
-// on the output).
+// the options of the other kernels (a soft cap of the scores; a sink in the softmax's denominator, of score 0 or of a score per head;
+// a gate per head on the output).
 //
 // The scheme is attention_mma.cu's: one thread block per (request, key/value head, tile of query rows, split of the keys);
 // the rows of a tile are the pairs (token, query head of the kv head's group), token-major; W warps of 16 rows each; key and
@@ -24,7 +24,7 @@ attention_mma_any_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
                          int n_kv, int d, int dv, float scale_log2, int window, __nv_bfloat16* __restrict__ out,
                          float* __restrict__ part_o, float* __restrict__ part_lse, int num_splits, int sink,
                          const float* __restrict__ sink_scores,
-                         const __nv_bfloat16* __restrict__ gate, int gate_ld, int chunk, int n_v) {
+                         const __nv_bfloat16* __restrict__ gate, int gate_ld, int chunk, int n_v, float cap_log2) {
   grid_dependency_wait();
   grid_dependency_launch();
   constexpr int BM = 16 * W, THREADS = 32 * W;
@@ -165,6 +165,13 @@ attention_mma_any_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
       }
     }
 
+    if (cap_log2 > 0.f) {                  // scores under a soft cap: from here on their tanh, scaled by the cap
+#pragma unroll
+      for (int n = 0; n < BN / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc_s[n][e] = capped_score(acc_s[n][e], cap_log2);
+    }
+
     // ---- mask and online softmax (scores are scaled inside the exponent)
     float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -289,7 +296,7 @@ int launch_attention_any(const void* q, const void* k_pool, const void* v_pool, 
                          const int* query_start, const int* context_lens, int page_size, int n_q, int n_kv, int d, int dv,
                          float scale, int window, void* out, float* part_o, float* part_lse, int num_splits, int n_requests,
                          int max_query_len, int n_tokens, int sink, const float* sink_scores, const void* gate, int gate_ld, int first_token,
-                         int chunk, int n_v, cudaStream_t stream) {
+                         int chunk, int n_v, float softcap, cudaStream_t stream) {
   constexpr int BM = 16 * W;
   const size_t smem = (size_t)(BM * (d + 8) + 2 * BN * (d + 8) + 2 * BN * (dv + 8)) * sizeof(__nv_bfloat16) + 4 * BN * sizeof(long long);
   auto kernel = attention_mma_any_kernel<W, BN>;
@@ -306,8 +313,10 @@ int launch_attention_any(const void* q, const void* k_pool, const void* v_pool, 
              "attention (any head size): grid %lld x %d x %lld exceeds the launch limits", tiles, n_kv, (long long)n_requests * num_splits);
   dim3 grid((unsigned)tiles, n_kv, n_requests * num_splits);
   ms::launch(kernel, grid, W * 32, smem, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool,
-             block_tables, table_stride, query_start, context_lens, page_size, n_q, n_kv, d, dv, scale * 1.4426950408889634f, window,
-             (__nv_bfloat16*)out, part_o, part_lse, num_splits, sink, sink_scores, (const __nv_bfloat16*)gate, gate_ld, chunk, n_v);
+             block_tables, table_stride, query_start, context_lens, page_size, n_q, n_kv, d, dv,
+             (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window,
+             (__nv_bfloat16*)out, part_o, part_lse, num_splits, sink, sink_scores, (const __nv_bfloat16*)gate, gate_ld, chunk, n_v,
+             softcap > 0.f ? 2.f * scale / softcap * 1.4426950408889634f : 0.f);
   MS_CHECK_LAUNCH("attention_mma_any");
   if (num_splits > 1) {
     const size_t skip = (size_t)first_token * n_q;
@@ -345,13 +354,13 @@ MS_EXPORT int ms_attention_mma_any_splits(int n_requests, int n_kv, int n_q, int
 
 // Arguments as ms_paged_attention_mma, with the value heads' size dv: q [n_tokens, n_q, d], key pool [pages, n_kv, page_size, d],
 // value pool [pages, n_v, page_size, dv] (n_v a divisor of n_kv: key head g reads value head g % n_v), out [n_tokens, n_q, dv];
-// part_o [n_tokens * n_q * num_splits * dv].
+// part_o [n_tokens * n_q * num_splits * dv].  softcap c > 0: a scaled score s becomes c tanh(s / c).
 MS_EXPORT int ms_paged_attention_mma_any(const void* q, const void* k_pool, const void* v_pool, const int* block_tables,
                                          int table_stride, const int* query_start, const int* context_lens, int page_size,
                                          int n_q, int n_kv, int d, int dv, float scale, int window, void* out, float* part_o,
                                          float* part_lse, int num_splits, int n_requests, int max_query_len, int n_tokens,
                                          int sink, const float* sink_scores, const void* gate, int gate_ld, int first_token, int chunk,
-                                         int n_v, cudaStream_t stream) {
+                                         int n_v, float softcap, cudaStream_t stream) {
   if (n_tokens == 0 || n_requests == 0) return 0;
   MS_REQUIRE(ms_attention_mma_any_supports(d, dv), "attention (any head size): sizes %d and %d are not multiples of 16 up to %d", d, dv, kAnyMax);
   MS_REQUIRE(n_kv > 0 && n_q % n_kv == 0, "attention: %d query heads are not a multiple of %d key/value heads", n_q, n_kv);
@@ -363,8 +372,8 @@ MS_EXPORT int ms_paged_attention_mma_any(const void* q, const void* k_pool, cons
   if (small)
     return launch_attention_any<1, 32>(q, k_pool, v_pool, block_tables, table_stride, query_start, context_lens, page_size, n_q, n_kv, d,
                                        dv, scale, window, out, part_o, part_lse, num_splits, n_requests, max_query_len, n_tokens, sink,
-                                       sink_scores, gate, gate_ld, first_token, chunk, n_v, stream);
+                                       sink_scores, gate, gate_ld, first_token, chunk, n_v, softcap, stream);
   return launch_attention_any<4, 64>(q, k_pool, v_pool, block_tables, table_stride, query_start, context_lens, page_size, n_q, n_kv, d, dv,
                                      scale, window, out, part_o, part_lse, num_splits, n_requests, max_query_len, n_tokens, sink, sink_scores, gate,
-                                     gate_ld, first_token, chunk, n_v, stream);
+                                     gate_ld, first_token, chunk, n_v, softcap, stream);
 }

@@ -55,14 +55,14 @@ struct Layout {
   static constexpr size_t TOTAL = (size_t)Q_BYTES + (size_t)(K_STAGES + V_STAGES) * TILE_BYTES + 1024;
 };
 
-template <int D>
+template <int D, bool CAPPED>
 __global__ void __launch_bounds__(THREADS, 1)
 attention_turns_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_out,
                        const int* __restrict__ block_tables, int table_stride,
                        const int* __restrict__ query_start, const int* __restrict__ context_lens, int page_size, int n_q,
                        int n_kv, float scale_log2, int window, __nv_bfloat16* __restrict__ out, int* __restrict__ error_flag,
-                       int sink, const float* __restrict__ sink_scores, const __nv_bfloat16* __restrict__ gate, int gate_ld) {
+                       int sink, const float* __restrict__ sink_scores, const __nv_bfloat16* __restrict__ gate, int gate_ld, float cap_log2) {
   using L = Layout<D>;
   extern __shared__ unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -261,6 +261,10 @@ attention_turns_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 #pragma unroll
         for (int c = 0; c < BN; c += 32) tmem_load_32_nowait(s_addr + c, *reinterpret_cast<float(*)[32]>(&v[c]));
         tmem_load_wait();
+        if (CAPPED) {                    // scores under a soft cap: from here on their tanh, scaled by the cap
+#pragma unroll
+          for (int i = 0; i < BN; ++i) v[i] = capped_score(v[i], cap_log2);
+        }
         // eight independent partial maxima (and sums below): a single running value would chain 128 operations
         float part_max[8];
 #pragma unroll
@@ -429,11 +433,11 @@ static bool encode(CUtensorMap* map, int rank, const void* base, const cuuint64_
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int D>
+template <int D, bool CAPPED>
 int launch(const void* q, const void* k_pool, const void* v_pool, int n_pages, const int* block_tables, int table_stride,
            const int* query_start, const int* context_lens, int page_size, int n_q, int n_kv, float scale, int window,
            void* out, int n_requests, int max_query_len, int n_tokens, int* error_flag, int sink, const float* sink_scores, const void* gate, int gate_ld,
-           cudaStream_t stream) {
+           float softcap, cudaStream_t stream) {
   const int group = n_q / n_kv;
   CUtensorMap map_q, map_k, map_v, map_out;
   {
@@ -450,7 +454,7 @@ int launch(const void* q, const void* k_pool, const void* v_pool, int n_pages, c
     MS_REQUIRE(encode(&map_k, 2, k_pool, dims, strides, box) && encode(&map_v, 2, v_pool, dims, strides, box),
                "attention_turns: tensor map of the cache pools failed");
   }
-  auto kernel = attention_turns_kernel<D>;
+  auto kernel = attention_turns_kernel<D, CAPPED>;
   const size_t smem = Layout<D>::TOTAL;
   static bool configured = false;
   if (!configured) {
@@ -462,8 +466,9 @@ int launch(const void* q, const void* k_pool, const void* v_pool, int n_pages, c
   MS_REQUIRE(tiles <= 65535 && n_requests <= 65535, "attention_turns: grid exceeds the launch limits");
   dim3 grid(n_kv, (unsigned)tiles, n_requests);
   cudaError_t e = ms::launch(kernel, grid, dim3(THREADS), smem, stream, map_q, map_k, map_v, map_out, block_tables, table_stride,
-                             query_start, context_lens, page_size, n_q, n_kv, scale * 1.4426950408889634f, window,
-                             (__nv_bfloat16*)out, error_flag, sink, sink_scores, (const __nv_bfloat16*)gate, gate_ld);
+                             query_start, context_lens, page_size, n_q, n_kv, (CAPPED ? softcap : scale) * 1.4426950408889634f, window,
+                             (__nv_bfloat16*)out, error_flag, sink, sink_scores, (const __nv_bfloat16*)gate, gate_ld,
+                             CAPPED ? 2.f * scale / softcap * 1.4426950408889634f : 0.f);
   if (e != cudaSuccess) MS_FAIL("attention_turns: launch failed: %s", cudaGetErrorString(e));
   return 0;
 }
@@ -473,24 +478,24 @@ int launch(const void* q, const void* k_pool, const void* v_pool, int n_pages, c
 
 using namespace ms;
 
-// Arguments and sizes as for ms_paged_attention_tcgen05 (ms_attention_tcgen05_supports answers for both), and two options:
+// Arguments and sizes as for ms_paged_attention_tcgen05 (ms_attention_tcgen05_supports answers for both), and three options:
 // sink != 0 adds exp(0), or exp(sink_scores[head]) (float32 [n_q], not null), to every row's softmax denominator (a key without
-// a value); gate (bfloat16 logits,
+// a value); softcap c > 0 turns a scaled score s into c tanh(s / c); gate (bfloat16 logits,
 // gate[token * gate_ld + head], or null) multiplies each head's output by the sigmoid of its logit as it is stored.
 MS_EXPORT int ms_paged_attention_turns(const void* q, const void* k_pool, const void* v_pool, int n_pages,
                                        const int* block_tables, int table_stride, const int* query_start,
                                        const int* context_lens, int page_size, int n_q, int n_kv, int d, float scale,
                                        int window, void* out, int n_requests, int max_query_len, int n_tokens,
-                                       int* error_flag, int sink, const float* sink_scores, const void* gate, int gate_ld, cudaStream_t stream) {
+                                       int* error_flag, int sink, const float* sink_scores, const void* gate, int gate_ld, float softcap,
+                                       cudaStream_t stream) {
   if (n_tokens == 0 || n_requests == 0) return 0;
   const int group = n_kv > 0 && n_q % n_kv == 0 ? n_q / n_kv : 0;
   MS_REQUIRE((d == 64 || d == 128) && group > 0 && group <= 128 && 128 % group == 0 && page_size >= 8 && page_size <= 128 &&
              128 % page_size == 0,
              "attention_turns: head size %d, %d/%d heads, page size %d are not taken by this kernel", d, n_q, n_kv, page_size);
   MS_REQUIRE(error_flag != nullptr, "attention_turns: an error flag on the device is required");
-  if (d == 128)
-    return t5c::launch<128>(q, k_pool, v_pool, n_pages, block_tables, table_stride, query_start, context_lens, page_size,
-                            n_q, n_kv, scale, window, out, n_requests, max_query_len, n_tokens, error_flag, sink, sink_scores, gate, gate_ld, stream);
-  return t5c::launch<64>(q, k_pool, v_pool, n_pages, block_tables, table_stride, query_start, context_lens, page_size, n_q,
-                         n_kv, scale, window, out, n_requests, max_query_len, n_tokens, error_flag, sink, sink_scores, gate, gate_ld, stream);
+  auto launch = d == 128 ? (softcap > 0.f ? t5c::launch<128, true> : t5c::launch<128, false>)
+                         : (softcap > 0.f ? t5c::launch<64, true> : t5c::launch<64, false>);
+  return launch(q, k_pool, v_pool, n_pages, block_tables, table_stride, query_start, context_lens, page_size, n_q, n_kv, scale, window,
+                out, n_requests, max_query_len, n_tokens, error_flag, sink, sink_scores, gate, gate_ld, softcap, stream);
 }

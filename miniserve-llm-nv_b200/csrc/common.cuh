@@ -101,6 +101,22 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   return total;
 }
 
+// Activations of gated feed-forwards: silu(g) u, the clamped form (see clamped_times), gelu_tanh(g) u.
+enum : int { kGateSilu = 0, kGateClamped = 1, kGateGelu = 2 };
+
+// gelu_tanh(z) = z/2 (1 + tanh y) = z sigmoid(2 y) with y = sqrt(2 / pi) (z + 0.044715 z^3).
+__device__ __forceinline__ float gelu_tanh_exponent(float z) { return 1.5957691216057308f * (z + 0.044715f * z * z * z); }
+
+// A raw score q . k under a soft cap c (score = c tanh(s / c), s = scale q . k): tanh(pre * raw) with pre = scale / c; what
+// follows multiplies by c.  tanh x = 1 - 2 / (1 + e^(2 x)), whose absolute error is about 2^-23 whatever x is (an infinite e^(2 x)
+// gives 1, a vanished one -1); twice_pre_log2 = 2 pre log2(e).
+__device__ __forceinline__ float capped_score(float raw, float twice_pre_log2) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * twice_pre_log2));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return fmaf(-2.f, r, 1.f);
+}
+
 // A sink in a row's softmax: one more term 2^sink2 of the denominator that has no value (sink2: its score times log2 e).  `top` is the
 // row's running maximum in base 2 (meaningless where nothing was seen: `seen` false) and `l` its sum relative to 2^top; both
 // become those of the row with the sink.  Returns the factor of what was accumulated relative to the old maximum.

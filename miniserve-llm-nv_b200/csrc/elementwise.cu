@@ -196,7 +196,8 @@ __global__ void qk_norm_rope_append_kernel(const T* __restrict__ qkv, const int*
 // ---------------------------------------------------------------- gated activation
 // out[n, c] = silu(gate_up[n, c]) * gate_up[n, inter + c]
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total, float limit) {
+__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total, int activation,
+                                float limit) {
   grid_dependency_wait();
   grid_dependency_launch();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -205,7 +206,8 @@ __global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ o
   const int c = (int)(i % inter);
   const float g = to_float(gate_up[n * 2 * inter + c]);
   const float u = to_float(gate_up[n * 2 * inter + inter + c]);
-  out[i] = from_float<T>(limit > 0.f ? clamped_times(g, u, limit) : g / (1.0f + expf(-g)) * u);
+  out[i] = from_float<T>(activation == kGateClamped ? clamped_times(g, u, limit)
+                         : activation == kGateGelu ? gelu_times<float>(g, u) : g / (1.0f + expf(-g)) * u);
 }
 
 }  // namespace ms
@@ -330,25 +332,27 @@ MS_EXPORT int ms_qk_norm_rope_append(const void* qkv, int dtype, const int* slot
 }
 
 // paired != 0: gate and up columns alternate in blocks of eight (inter must be a multiple of 8 then).
-// limit > 0: the clamped gated activation in place of silu(gate) * up.
-MS_EXPORT int ms_silu_mul(const void* gate_up, int dtype, void* out, int n_tokens, int inter, int paired, float limit,
-                          cudaStream_t stream) {
+// activation: 0 silu(gate) * up, 1 the clamped gated activation with `limit`, 2 gelu_tanh(gate) * up.
+MS_EXPORT int ms_silu_mul(const void* gate_up, int dtype, void* out, int n_tokens, int inter, int paired, int activation,
+                          float limit, cudaStream_t stream) {
   const size_t total = (size_t)n_tokens * inter;
   if (total == 0) return 0;
+  MS_REQUIRE(activation >= kGateSilu && activation <= kGateGelu && (activation != kGateClamped || limit > 0.f),
+             "silu_mul: activation %d with limit %f", activation, limit);
   MS_REQUIRE(!paired || inter % 8 == 0, "silu_mul: paired columns need a multiple of 8 features, not %d", inter);
   if (inter % 8 == 0) {
     const size_t total8 = total / 8;
     const size_t blocks8 = (total8 + 255) / 256;
     MS_REQUIRE(blocks8 < 2147483647ULL, "silu_mul: %zu elements in one launch is too many", total);
     MS_DISPATCH(dtype, (ms::launch(silu_mul_vec_kernel<T>, (unsigned)blocks8, 256, 0, stream, (const T*)gate_up, (T*)out, inter,
-                                                                                    total8, paired, limit)));
+                                                                                    total8, paired, activation, limit)));
     MS_CHECK_LAUNCH("silu_mul");
     return 0;
   }
   const size_t blocks = (total + 255) / 256;
   MS_REQUIRE(blocks < 2147483647ULL, "silu_mul: %zu elements in one launch is too many", total);
   MS_DISPATCH(dtype, (ms::launch(silu_mul_kernel<T>, (unsigned)blocks, 256, 0, stream, (const T*)gate_up, (T*)out, inter,
-                                                                             total, limit)));
+                                                                             total, activation, limit)));
   MS_CHECK_LAUNCH("silu_mul");
   return 0;
 }

@@ -144,13 +144,15 @@ __global__ void postnorm_add_rmsnorm_vec_kernel(float* __restrict__ residual, co
 // bias (null: none): float32 [ld], the projection's bias column by column, added in float32 to every head as it is read.
 // value_heads: the projection and the value pool [page, value_heads, page_size, dv] hold that many value heads (a divisor of
 // n_kv: key heads that share values).
+// kept (null: none): [n, value_heads * dv], values handed along the depth of the model.  mixed == 0: it receives the token's values
+// (bias included); mixed != 0: the values become (1 - mix) v + mix kept in float32 before they are stored.
 template <typename T>
 __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, int q_col, int k_col, int v_col, int n_q, int n_kv,
                                    int d, int dv, const int* __restrict__ slots, const float* __restrict__ q_weight,
                                    const float* __restrict__ k_weight, float eps, const float2* __restrict__ cos_sin,
                                    int rotary_dim, T* __restrict__ k_pool, T* __restrict__ v_pool, int page_size,
                                    T* __restrict__ q_out, int n_tokens, int interleaved, const float* __restrict__ bias,
-                                   int value_heads) {
+                                   int value_heads, T* __restrict__ kept, int mixed, float mix) {
   grid_dependency_wait();
   grid_dependency_launch();
   extern __shared__ float prepare_smem[];
@@ -172,11 +174,22 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, int q_col
     weight = q_weight;
   } else {
     const int slot = slots[n];
-    if (slot < 0) return;
+    if (slot < 0 && !(kept && !mixed && head >= n_q + n_kv)) return;
     const int page = slot / page_size, offset = slot % page_size;
     if (head >= n_q + n_kv) {
       const int g = head - n_q - n_kv;
       src = row + v_col + g * dv;                        // (value_heads of them: key head g reads value head g % value_heads)
+      if (kept) {
+        T* handed = kept + ((size_t)n * value_heads + g) * dv;
+        dst = v_pool + (((size_t)page * value_heads + g) * page_size + offset) * dv;
+        for (int c = lane; c < dv; c += 32) {
+          float v = to_float(src[c]) + (bias ? bias[v_col + g * dv + c] : 0.f);
+          if (!mixed) handed[c] = from_float<T>(v);
+          else v = (1.f - mix) * v + mix * to_float(handed[c]);
+          if (slot >= 0) dst[c] = from_float<T>(v);
+        }
+        return;
+      }
       dst = v_pool + (((size_t)page * value_heads + g) * page_size + offset) * dv;
       if (bias) {
         const float* b = bias + v_col + g * dv;
@@ -425,12 +438,14 @@ MS_EXPORT int ms_postnorm_add_rmsnorm(float* residual, const void* delta, int dt
 MS_EXPORT int ms_qkv_prepare(const void* proj, int dtype, int ld, int q_col, int k_col, int v_col, int n_q, int n_kv, int d,
                              int dv, const int* slots, const float* q_weight, const float* k_weight, float eps,
                              const float* cos_sin, int rotary_dim, void* k_pool, void* v_pool, int page_size, void* q_out,
-                             int n_tokens, int interleaved, const float* bias, int value_heads, cudaStream_t stream) {
+                             int n_tokens, int interleaved, const float* bias, int value_heads, void* kept, int mixed, float mix,
+                             cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   MS_REQUIRE(d > 0 && d <= 1024 && dv > 0, "qkv_prepare: head sizes %d and %d", d, dv);
   MS_REQUIRE(rotary_dim >= 0 && rotary_dim <= d && rotary_dim % 2 == 0,
              "qkv_prepare: rotary size %d must be even and at most the head size %d", rotary_dim, d);
   MS_REQUIRE(page_size > 0, "qkv_prepare: page size must be positive, got %d", page_size);
+  MS_REQUIRE(kept == nullptr || k_col >= 0, "qkv_prepare: values handed along need values of the layer's own");
   MS_REQUIRE(k_col < 0 || (v_col >= 0 && slots && k_pool && v_pool), "qkv_prepare: keys and values need their columns, slots and pools");
   MS_REQUIRE(k_col < 0 || (value_heads >= 1 && n_kv % value_heads == 0), "qkv_prepare: %d value heads for %d key heads", value_heads, n_kv);
   const int warps = 4;
@@ -440,7 +455,8 @@ MS_EXPORT int ms_qkv_prepare(const void* proj, int dtype, int ld, int q_col, int
   const size_t smem = (size_t)warps * d * sizeof(float);
   MS_EG_DISPATCH(dtype, (ms::launch(qkv_prepare_kernel<T>, (unsigned)blocks, warps * 32, smem, stream, (const T*)proj, ld, q_col,
                                     k_col, v_col, n_q, n_kv, d, dv, slots, q_weight, k_weight, eps, (const float2*)cos_sin,
-                                    rotary_dim, (T*)k_pool, (T*)v_pool, page_size, (T*)q_out, n_tokens, interleaved, bias, value_heads > 0 ? value_heads : n_kv)));
+                                    rotary_dim, (T*)k_pool, (T*)v_pool, page_size, (T*)q_out, n_tokens, interleaved, bias, value_heads > 0 ? value_heads : n_kv,
+                                    (T*)kept, mixed, mix)));
   MS_CHECK_LAUNCH("qkv_prepare");
   return 0;
 }

@@ -314,9 +314,21 @@ __device__ __forceinline__ float clamped_times(float gate, float up, float limit
   return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
 
+// gelu_tanh(g) * u, the exponential and the division as in silu_times.
+template <typename T>
+__device__ __forceinline__ float gelu_times(float g, float u) {
+  const float y = gelu_tanh_exponent(g);
+  if (sizeof(T) == 2) {
+    const float e = __expf(-fabsf(y));
+    const float r = __fdividef(1.0f, 1.0f + e);
+    return g * (y >= 0.f ? r : e * r) * u;
+  }
+  return g / (1.0f + expf(-y)) * u;
+}
+
 template <typename T>
 __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total8, int paired,
-                                    float limit) {
+                                    int activation, float limit) {
   grid_dependency_wait();
   grid_dependency_launch();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -336,7 +348,10 @@ __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict
   const Vec8 u = load8(row + (paired ? 2 * c + 8 : inter + c));
   Vec8 y;
 #pragma unroll
-  for (int e = 0; e < 8; ++e) y.v[e] = limit > 0.f ? clamped_times(g.v[e], u.v[e], limit) : silu_times<T>(g.v[e], u.v[e]);
+  for (int e = 0; e < 8; ++e) {
+    y.v[e] = activation == kGateClamped ? clamped_times(g.v[e], u.v[e], limit)
+             : activation == kGateGelu  ? gelu_times<T>(g.v[e], u.v[e]) : silu_times<T>(g.v[e], u.v[e]);
+  }
   store8(out + n * inter + c, y);
 }
 

@@ -11,7 +11,7 @@
 //   ms_relu_square      x = max(x, 0)^2 in place
 //   ms_router_choose    another way to route: scores are the softmax over ALL router outputs, a correction is added for the
 //                       choice only, the outputs form groups of which only the best can be chosen from, and the weights are
-//                       the chosen scores as they are
+//                       the chosen scores as they are, or normalized and scaled
 //   ms_clamped_glu      out = g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit) for
 //                       alternating (gate, up) columns; the same activation is an epilogue of ms_expert_linear
 //
@@ -144,13 +144,16 @@ __global__ void router_select_kernel(const float* __restrict__ all_logits, int e
 }
 
 // One warp per token.  scores = softmax over the first `total` logits of the row; choice = score + correction; the
-// outputs form `group_count` equal groups of neighbours, a group's score is its largest choice score, and only members of
+// outputs form `group_count` equal groups of neighbours, a group's score is its largest choice score (group_two: the sum of its
+// two largest), and only members of
 // the `group_keep` best groups (ties: the lower group) can be chosen; the `top` largest choice scores among those are
-// taken one after the other (ties: the lower index); weights are the taken outputs' scores, not renormalised.  A choice
+// taken one after the other (ties: the lower index); weights are the taken outputs' scores as they are, or, normalize >= 0, divided
+// by (their sum + normalize), and then times weight_scale.  A choice
 // score that is not a number counts as the smallest, so that every id written is a valid one.
 __global__ void router_choose_kernel(const float* __restrict__ all_logits, int ld, int total, int top,
                                      const float* __restrict__ correction, int group_count, int group_keep,
-                                     int* __restrict__ ids, float* __restrict__ weights, int n_tokens, int sigmoid_scores) {
+                                     int* __restrict__ ids, float* __restrict__ weights, int n_tokens, int sigmoid_scores,
+                                     int group_two, float normalize, float weight_scale) {
   grid_dependency_wait();
   grid_dependency_launch();
   extern __shared__ float select_smem[];
@@ -184,9 +187,13 @@ __global__ void router_choose_kernel(const float* __restrict__ all_logits, int l
   const int per_group = total / group_count;
   if (group_keep < group_count) {
     for (int g = lane; g < group_count; g += 32) {
-      float best = -INFINITY;
-      for (int i = 0; i < per_group; ++i) best = fmaxf(best, choice[g * per_group + i]);
-      group_best[g] = best;
+      float best = -INFINITY, next = -INFINITY;
+      for (int i = 0; i < per_group; ++i) {
+        const float c = choice[g * per_group + i];
+        next = fmaxf(next, fminf(best, c));
+        best = fmaxf(best, c);
+      }
+      group_best[g] = group_two && per_group > 1 ? best + next : best;
     }
     __syncwarp();
     // a group is kept if fewer than `group_keep` groups come before it (a larger score, or the same with a lower index)
@@ -199,6 +206,7 @@ __global__ void router_choose_kernel(const float* __restrict__ all_logits, int l
     }
     __syncwarp();
   }
+  float taken = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int best_e = 0x7fffffff;
@@ -216,8 +224,13 @@ __global__ void router_choose_kernel(const float* __restrict__ all_logits, int l
       ids[(size_t)n * top + k] = best_e;
       weights[(size_t)n * top + k] = score[best_e];
       choice[best_e] = -INFINITY;
+      taken += score[best_e];
     }
     __syncwarp();
+  }
+  if (lane == 0 && (normalize >= 0.f || weight_scale != 1.f)) {
+    const float factor = normalize >= 0.f ? taken + normalize : 1.f;
+    for (int k = 0; k < top; ++k) weights[(size_t)n * top + k] = weights[(size_t)n * top + k] / factor * weight_scale;
   }
 }
 
@@ -576,9 +589,12 @@ MS_EXPORT int ms_router_topk(const void* x, int dtype, const float* weight, cons
 // The router whose scores are the softmax over all outputs (sigmoid_scores: the sigmoid of each output).  weight float32 [rows, width] with rows >= total: the first
 // `total` rows are the router's outputs, further rows ride along (their logits are left in `logits` for the caller);
 // bias [rows] or null; correction float32 [total] or null; logits float32 [n_tokens, rows]; ids, weights [n_tokens, top].
+// group_two: a group's score is the sum of its two largest choice scores instead of the largest; normalize >= 0: the weights are
+// divided by (their sum + normalize); weight_scale multiplies them.
 MS_EXPORT int ms_router_choose(const void* x, int dtype, const float* weight, const float* bias, int width, int rows,
                                int total, int top, const float* correction, int group_count, int group_keep, float* logits,
-                               int* ids, float* weights, int n_tokens, int sigmoid_scores, cudaStream_t stream) {
+                               int* ids, float* weights, int n_tokens, int sigmoid_scores, int group_two, float normalize,
+                               float weight_scale, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   MS_REQUIRE(total > 0 && rows >= total, "router_choose: %d outputs in %d rows", total, rows);
   MS_REQUIRE(group_count > 0 && total % group_count == 0 && group_keep >= 1 && group_keep <= group_count,
@@ -590,7 +606,7 @@ MS_EXPORT int ms_router_choose(const void* x, int dtype, const float* weight, co
   const size_t smem = (size_t)warps * (2 * total + group_count) * sizeof(float);
   MS_REQUIRE(smem <= 48 * 1024, "router_choose: %d outputs need %zu bytes of shared memory", total, smem);
   ms::launch(router_choose_kernel, (n_tokens + warps - 1) / warps, warps * 32, smem, stream, (const float*)logits, rows, total, top,
-             correction, group_count, group_keep, ids, weights, n_tokens, sigmoid_scores);
+             correction, group_count, group_keep, ids, weights, n_tokens, sigmoid_scores, group_two, normalize, weight_scale);
   MS_CHECK_LAUNCH("router_choose: selection");
   return 0;
 }

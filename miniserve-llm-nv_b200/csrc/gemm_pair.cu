@@ -95,13 +95,15 @@ struct Fold {
   int norm_dtype;
   float* out_partials;          // [column tiles, M], residual epilogue
   float* residual;              // [M, N], residual epilogue
-  float gate_limit;             // gated epilogue: 0 for silu(gate) * up, else the limit of the clamped activation
+  int activation;               // gated epilogue: kGateSilu, kGateClamped (with gate_limit) or kGateGelu
+  float gate_limit;
 };
 
 
 using wide::round_bf16;
 using wide::clamped_times;
 using wide::gated_times;
+using wide::gelu_times;
 using wide::silu_times;
 
 __device__ __forceinline__ void tma_store_2d(const CUtensorMap* map, const void* smem_src, int x, int y) {
@@ -138,7 +140,7 @@ __device__ __forceinline__ uint4 pack8(const float* v) {
   return packed;
 }
 
-template <int STAGES, int EPILOGUE, typename OutT, bool WIDE, bool CLAMPED>
+template <int STAGES, int EPILOGUE, typename OutT, bool WIDE, int ACTIVATION>
 __global__ void __launch_bounds__(threads(EPILOGUE), 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                  const __grid_constant__ CUtensorMap map_out, const __grid_constant__ CUtensorMap map_residual,
@@ -475,7 +477,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
                   const float g = round_bf16(v[16 * h + j] * scale), u = round_bf16(v[16 * h + 8 + j] * scale);
-                  r[j] = CLAMPED ? clamped_times(g, u, fold.gate_limit) : silu_times(g, u);
+                  r[j] = ACTIVATION == kGateClamped ? clamped_times(g, u, fold.gate_limit) : ACTIVATION == kGateGelu ? gelu_times(g, u) : silu_times(g, u);
                 }
                 *swizzled_piece(buffer, lane, 2 * part + h) = pack8(r);
               }
@@ -515,7 +517,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
             OutT* dst = out + (size_t)row * (N / 2) + col / 2;
 #pragma unroll
             for (int i = 0; i < 16; ++i)
-              if (col + 16 * (i >> 3) < N) dst[i] = from_float<OutT>(gated_times(round_bf16(v[16 * (i >> 3) + (i & 7)]), round_bf16(v[16 * (i >> 3) + 8 + (i & 7)]), fold.gate_limit));
+              if (col + 16 * (i >> 3) < N) dst[i] = from_float<OutT>(gated_times(round_bf16(v[16 * (i >> 3) + (i & 7)]), round_bf16(v[16 * (i >> 3) + 8 + (i & 7)]), ACTIVATION, fold.gate_limit));
           } else if (EPILOGUE == EPI_ADD_F32) {
             float* dst = reinterpret_cast<float*>(out) + (size_t)row * N + col;
 #pragma unroll
@@ -585,7 +587,7 @@ static bool out_map(CUtensorMap* map, void* base, int rows, int cols, bool float
   return true;
 }
 
-template <int STAGES, int EPILOGUE, typename OutT, bool WIDE = false, bool CLAMPED = false>
+template <int STAGES, int EPILOGUE, typename OutT, bool WIDE = false, int ACTIVATION = kGateSilu>
 int launch(const void* X, const void* W, void* out, int M, int N, int K, const Fold& fold, float* residual, int* error_flag,
            cudaStream_t stream, const Heads& heads = Heads{}) {
   CUtensorMap map_x, map_w, map_out, map_residual;
@@ -602,7 +604,7 @@ int launch(const void* X, const void* W, void* out, int M, int N, int K, const F
                "gemm_pair: the residual epilogue wants N %d a multiple of 8 and 16-byte aligned matrices", N);
     MS_REQUIRE(out_map(&map_residual, residual, M, N, true), "gemm_pair: cuTensorMapEncodeTiled failed for the residual stream");
   }
-  auto kernel = gemm_pair_kernel<STAGES, EPILOGUE, OutT, WIDE, CLAMPED>;
+  auto kernel = gemm_pair_kernel<STAGES, EPILOGUE, OutT, WIDE, ACTIVATION>;
   const size_t smem = (size_t)STAGES * (WIDE ? 3 : 2) * HALF * BK * 2 + read_warps(EPILOGUE) * warp_bytes(EPILOGUE) + 1024;
   static bool configured = false;
   if (!configured) {
@@ -649,8 +651,8 @@ using namespace ms;
 //   epilogue 0: out [M, N] stored as bfloat16 (out_dtype 1) or float32 (out_dtype 0);
 //   epilogue 1: added in place into the float32 matrix out [M, N];
 //   epilogue 2: W holds eight gate rows, then the same eight up rows, and so on (N a multiple of 16);
-//               out [M, N / 2] bfloat16 = silu(gate) * up, or, with gate_limit > 0, g sigmoid(1.702 g) (u + 1) with
-//               g = min(gate, gate_limit) and u = clamp(up, -gate_limit, gate_limit);
+//               out [M, N / 2] bfloat16 = silu(gate) * up (activation 0), g sigmoid(1.702 g) (u + 1) with
+//               g = min(gate, gate_limit) and u = clamp(up, -gate_limit, gate_limit) (1), or gelu_tanh(gate) * up (2);
 //   epilogue 3: residual [M, N] float32 += the product, in place; out [M, N] bfloat16 = residual * norm_weight
 //               (norm_weight [N] of type norm_dtype); out_partials [ms_gemm_pair_column_tiles(N), M] float32
 //               receives the rows' sums of squares over each tile's columns (N a multiple of 8).
@@ -662,7 +664,8 @@ using namespace ms;
 // checks when it synchronises.
 MS_EXPORT int ms_gemm_pair(const void* X, const void* W, void* out, int out_dtype, int epilogue, int wide, int M, int N, int K,
                            const float* in_partials, int in_count, float eps, float* residual, const void* norm_weight,
-                           int norm_dtype, float* out_partials, float gate_limit, int* error_flag, cudaStream_t stream) {
+                           int norm_dtype, float* out_partials, int activation, float gate_limit, int* error_flag,
+                           cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
   MS_REQUIRE(K > 0 && K % 8 == 0, "gemm_pair: inner size %d is not a multiple of 8", K);
   MS_REQUIRE(((uintptr_t)X % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_pair: operands must be 16-byte aligned");
@@ -670,7 +673,7 @@ MS_EXPORT int ms_gemm_pair(const void* X, const void* W, void* out, int out_dtyp
   MS_REQUIRE(in_partials == nullptr || (in_count > 0 && (epilogue == pair::EPI_STORE || epilogue == pair::EPI_GATED)),
              "gemm_pair: row statistics go with the storing and the gated epilogue (count %d, epilogue %d)", in_count, epilogue);
   constexpr int STAGES = 6, STAGES_RESIDUAL = 5, STAGES_WIDE = 4;      // what fits beside the read-out warps' buffers
-  const pair::Fold fold{in_partials, in_count, eps, norm_weight, norm_dtype, out_partials, residual, gate_limit};
+  const pair::Fold fold{in_partials, in_count, eps, norm_weight, norm_dtype, out_partials, residual, activation, gate_limit};
   if (epilogue == pair::EPI_RESIDUAL) {
     MS_REQUIRE(out_dtype == MS_BF16 && residual != nullptr && norm_weight != nullptr && out_partials != nullptr &&
                (norm_dtype == MS_F32 || norm_dtype == MS_BF16),
@@ -684,9 +687,14 @@ MS_EXPORT int ms_gemm_pair(const void* X, const void* W, void* out, int out_dtyp
   }
   if (epilogue == pair::EPI_GATED) {
     MS_REQUIRE(out_dtype == MS_BF16 && N % 16 == 0, "gemm_pair: the gated epilogue stores bfloat16 and wants N %d a multiple of 16", N);
-    if (gate_limit > 0.f)
-      return wide ? pair::launch<STAGES_WIDE, pair::EPI_GATED, __nv_bfloat16, true, true>(X, W, out, M, N, K, fold, nullptr, error_flag, stream)
-                  : pair::launch<STAGES, pair::EPI_GATED, __nv_bfloat16, false, true>(X, W, out, M, N, K, fold, nullptr, error_flag, stream);
+    MS_REQUIRE(activation >= kGateSilu && activation <= kGateGelu && (activation != kGateClamped || gate_limit > 0.f),
+               "gemm_pair: activation %d with limit %f", activation, gate_limit);
+    if (activation == kGateClamped)
+      return wide ? pair::launch<STAGES_WIDE, pair::EPI_GATED, __nv_bfloat16, true, kGateClamped>(X, W, out, M, N, K, fold, nullptr, error_flag, stream)
+                  : pair::launch<STAGES, pair::EPI_GATED, __nv_bfloat16, false, kGateClamped>(X, W, out, M, N, K, fold, nullptr, error_flag, stream);
+    if (activation == kGateGelu)
+      return wide ? pair::launch<STAGES_WIDE, pair::EPI_GATED, __nv_bfloat16, true, kGateGelu>(X, W, out, M, N, K, fold, nullptr, error_flag, stream)
+                  : pair::launch<STAGES, pair::EPI_GATED, __nv_bfloat16, false, kGateGelu>(X, W, out, M, N, K, fold, nullptr, error_flag, stream);
     return wide ? pair::launch<STAGES_WIDE, pair::EPI_GATED, __nv_bfloat16, true>(X, W, out, M, N, K, fold, nullptr, error_flag, stream)
                 : pair::launch<STAGES, pair::EPI_GATED, __nv_bfloat16>(X, W, out, M, N, K, fold, nullptr, error_flag, stream);
   }
@@ -719,7 +727,7 @@ MS_EXPORT int ms_gemm_pair_qkv(const void* X, const void* W, void* q_out, int M,
   MS_REQUIRE(slots != nullptr && error_flag != nullptr, "gemm_pair_qkv: slots and an error flag on the device are required");
   MS_REQUIRE(weight_dtype == MS_F32 || weight_dtype == MS_BF16, "gemm_pair_qkv: unknown norm weight type code %d", weight_dtype);
   MS_REQUIRE(in_partials == nullptr || in_count > 0, "gemm_pair_qkv: row statistics of %d tiles", in_count);
-  const pair::Fold fold{in_partials, in_count, fold_eps, nullptr, 0, nullptr, nullptr, 0.f};
+  const pair::Fold fold{in_partials, in_count, fold_eps, nullptr, 0, nullptr, nullptr, kGateSilu, 0.f};
   const pair::Heads heads{slots, q_weight, k_weight, weight_dtype, eps, cos_sin, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool,
                           page_size, n_q, n_kv};
   return pair::launch<5, pair::EPI_QKV, __nv_bfloat16>(X, W, q_out, M, N, K, fold, nullptr, error_flag, stream, heads);

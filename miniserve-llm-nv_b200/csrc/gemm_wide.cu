@@ -82,7 +82,8 @@ struct Fold {
   int norm_dtype;
   __nv_bfloat16* x_next;         // [M, N]
   float* out_partials;           // [blocks][X_ROWS]
-  float gate_limit;              // gated mode: 0 for silu(gate) * up, else the limit of the clamped activation
+  int activation;                // gated mode: kGateSilu, kGateClamped (with gate_limit) or kGateGelu
+  float gate_limit;
 };
 
 struct Plan {
@@ -260,9 +261,9 @@ __device__ __forceinline__ void compute(const Consumer& c, const Plan& plan, con
       } else if (MODE == MODE_GATED) {
         const int feature = (group * TILES + c.warp) * 8 + r, features = N / 2;
         if (feature < features) {
-          if (t0 < M) out[(size_t)t0 * features + feature] = from_float<OutT>(gated_times(round_bf16(sum.x), round_bf16(sum.z), fold.gate_limit));
+          if (t0 < M) out[(size_t)t0 * features + feature] = from_float<OutT>(gated_times(round_bf16(sum.x), round_bf16(sum.z), fold.activation, fold.gate_limit));
           if (t0 + 1 < M)
-            out[(size_t)(t0 + 1) * features + feature] = from_float<OutT>(gated_times(round_bf16(sum.y), round_bf16(sum.w), fold.gate_limit));
+            out[(size_t)(t0 + 1) * features + feature] = from_float<OutT>(gated_times(round_bf16(sum.y), round_bf16(sum.w), fold.activation, fold.gate_limit));
         }
       } else {
         const int row = (group * TILES + c.warp) * 16 + r;
@@ -601,8 +602,8 @@ MS_EXPORT int ms_gemm_wide_blocks(int N, int K) {
 //   mode 0: out [M, N], bfloat16 (out_dtype 1) or float32 (0);
 //   mode 1: W holds a gated feed-forward's gate and up projections in blocks of sixteen rows (eight gate rows,
 //           then the up rows of the same eight features; N a multiple of 16); out [M, N / 2] bfloat16 =
-//           silu(gate) * up, or, with gate_limit > 0, g sigmoid(1.702 g) (u + 1) with g = min(gate, gate_limit) and
-//           u = clamp(up, -gate_limit, gate_limit).
+//           silu(gate) * up (activation 0), g sigmoid(1.702 g) (u + 1) with g = min(gate, gate_limit) and
+//           u = clamp(up, -gate_limit, gate_limit) (1), or gelu_tanh(gate) * up (2).
 // error_flag: one int on the device, zero before the first call; a kernel that gave up waiting writes a
 // non-zero code there (1, 4 copies; 2, 3 products), which the caller checks when it synchronises.
 //
@@ -613,7 +614,8 @@ MS_EXPORT int ms_gemm_wide_blocks(int N, int K) {
 //           float32 = sums of residual^2 over each block's columns; only for weights with ms_gemm_wide_supports == 2.
 MS_EXPORT int ms_gemm_wide(const void* X, const void* W, void* out, int out_dtype, int mode, int M, int N, int K,
                            const float* in_partials, int in_count, float eps, float* residual, const void* norm_weight,
-                           int norm_dtype, void* x_next, float* out_partials, float gate_limit, int* error_flag, cudaStream_t stream) {
+                           int norm_dtype, void* x_next, float* out_partials, int activation, float gate_limit, int* error_flag,
+                           cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
   wide::Fold fold = {};
   fold.in_partials = in_count > 0 ? in_partials : nullptr;
@@ -625,12 +627,15 @@ MS_EXPORT int ms_gemm_wide(const void* X, const void* W, void* out, int out_dtyp
   fold.norm_dtype = norm_dtype;
   fold.x_next = (__nv_bfloat16*)x_next;
   fold.out_partials = out_partials;
+  fold.activation = activation;
   fold.gate_limit = gate_limit;
   MS_REQUIRE(M <= wide::X_ROWS, "gemm_wide: %d rows; this kernel takes at most %d", M, wide::X_ROWS);
   MS_REQUIRE(K > 0 && K % 8 == 0, "gemm_wide: inner size %d is not a multiple of 8", K);
   MS_REQUIRE(((uintptr_t)X % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_wide: operands must be 16-byte aligned");
   MS_REQUIRE(error_flag != nullptr, "gemm_wide: an error flag on the device is required");
   if (mode == wide::MODE_GATED) {
+    MS_REQUIRE(activation >= kGateSilu && activation <= kGateGelu && (activation != kGateClamped || gate_limit > 0.f),
+               "gemm_wide: activation %d with limit %f", activation, gate_limit);
     MS_REQUIRE(N % 16 == 0 && out_dtype == MS_BF16, "gemm_wide: gated mode wants a multiple of 16 rows (%d) and bfloat16 results", N);
     return wide::launch<wide::MODE_GATED, __nv_bfloat16>(X, W, out, M, N, K, fold, error_flag, stream);
   }

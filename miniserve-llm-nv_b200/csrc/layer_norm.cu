@@ -1,8 +1,10 @@
-// Layer norm of the residual stream, and the kernel that hands the stream to a matrix product.
+// Layer norm and dynamic tanh of the residual stream, and the kernel that hands the stream to a matrix product.
 //
 //   ms_add_layernorm      pending outputs (or a vector) are added to the float32 stream, and the sum is layer-normed for the
 //                         sublayers that read it next: one output, or two with weights and biases of their own that share the
 //                         row's mean and deviation (a block whose mixer and feed-forward each have a norm of the same stream)
+//   ms_add_dynamic_tanh   pending outputs are added to the float32 stream, and the sum passes weight * tanh(alpha x) + bias entry by
+//                         entry: a norm without statistics, so nothing ties the entries of a row together
 //   ms_stream_to_columns  the stream with its pending outputs, rounded once to the compute type, as some columns of a wider
 //                         matrix (the input of a product over the stream and something beside it)
 //
@@ -150,6 +152,59 @@ __global__ void add_layernorm_vec_kernel(float* __restrict__ residual, const T* 
   }
 }
 
+// For output row k (source row r = rows ? rows[k] : k), entry by entry:
+//   x = residual[r] + (delta[r] + delta2[r])      (written back unless rows are gathered or nothing was added)
+//   out[k] = weight * tanh(alpha x) + bias, rounded once to T
+// PER entries a thread (8: sixteen-byte accesses, hidden % 8 == 0; 1 otherwise).  A thread keeps its columns
+// from row to row: grid.x blocks cover the columns, grid.y strides over the rows, so weights and biases are fetched once, while
+// the kernel before ends.
+template <typename T, int PER>
+__global__ void __launch_bounds__(128)
+add_dynamic_tanh_kernel(float* __restrict__ residual, const T* __restrict__ delta, const T* __restrict__ delta2, float alpha,
+                        const float* __restrict__ weight, const float* __restrict__ bias, const int* __restrict__ rows,
+                        T* __restrict__ out, int n_out, int hidden) {
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * PER;
+  Vec8 w, b;
+  if (c < hidden) {
+    if (PER == 8) {
+      w = load8(weight + c), b = load8(bias + c);
+    } else {
+      w.v[0] = weight[c], b.v[0] = bias[c];
+    }
+  }
+  grid_dependency_wait();
+  grid_dependency_launch();
+  if (c >= hidden) return;
+  for (int k = blockIdx.y; k < n_out; k += gridDim.y) {
+    const size_t at = (size_t)(rows ? rows[k] : k) * hidden + c;
+    Vec8 x, y;
+    if (PER == 8) {
+      x = load8(residual + at);
+      if (delta) {
+        Vec8 d = load8(delta + at);
+        if (delta2) {
+          const Vec8 d2 = load8(delta2 + at);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) d.v[e] += d2.v[e];
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x.v[e] += d.v[e];
+        if (rows == nullptr) store8(residual + at, x);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y.v[e] = w.v[e] * tanhf(alpha * x.v[e]) + b.v[e];
+      store8(out + (size_t)k * hidden + c, y);
+    } else {
+      float v = residual[at];
+      if (delta) {
+        v += delta2 ? to_float(delta[at]) + to_float(delta2[at]) : to_float(delta[at]);
+        if (rows == nullptr) residual[at] = v;
+      }
+      out[(size_t)k * hidden + c] = from_float<T>(w.v[0] * tanhf(alpha * v) + b.v[0]);
+    }
+  }
+}
+
 // out[n, col + c] = residual[n, c] + (delta[n, c] + delta2[n, c]), rounded once to T; `pieces`: groups of eight a row (0: one
 // number a thread).
 template <typename T>
@@ -218,6 +273,32 @@ MS_EXPORT int ms_add_layernorm(float* residual, const void* delta, const void* d
   MS_LN_DISPATCH(dtype, (ms::launch(add_layernorm_kernel<T>, n_out, threads, 0, stream, residual, (const T*)delta, (const T*)delta2,
                                     vector, weight, bias, weight2, bias2, weight_dtype, eps, rows, (T*)out, (T*)out2, hidden)));
   MS_CHECK_LAUNCH("add_layernorm");
+  return 0;
+}
+
+// residual float32 [rows, hidden]; delta, delta2 (delta2 only with delta) [rows, hidden] and out [n_out, hidden] of type `dtype`;
+// weight, bias float32 [hidden]; rows int32 [n_out] or null (then n_out rows in place, and the residual receives the sum).
+MS_EXPORT int ms_add_dynamic_tanh(float* residual, const void* delta, const void* delta2, int dtype, float alpha, const float* weight,
+                                  const float* bias, const int* rows, void* out, int n_out, int hidden, cudaStream_t stream) {
+  if (n_out == 0) return 0;
+  MS_REQUIRE(hidden > 0, "add_dynamic_tanh: width %d", hidden);
+  MS_REQUIRE(delta2 == nullptr || delta != nullptr, "add_dynamic_tanh: a second output without a first");
+  auto aligned = [](const void* p) { return reinterpret_cast<size_t>(p) % 16 == 0; };
+  const bool wide = hidden % 8 == 0 && aligned(residual) && aligned(delta) && aligned(delta2) && aligned(weight) && aligned(bias) && aligned(out);
+  const int items = wide ? hidden / 8 : hidden;
+  int threads = items >= 128 ? 128 : ((items + 31) / 32) * 32;
+  const int column_blocks = (items + threads - 1) / threads;
+  // about sixteen blocks of 128 threads a multiprocessor stride over the rows
+  long long row_blocks = 148LL * 16 / column_blocks;
+  if (row_blocks < 1) row_blocks = 1;
+  if (row_blocks > n_out) row_blocks = n_out;
+  dim3 grid(column_blocks, (unsigned)row_blocks);
+#define MS_DYNAMIC_TANH(PER)                                                                                                   \
+  MS_LN_DISPATCH(dtype, (ms::launch(add_dynamic_tanh_kernel<T, PER>, grid, threads, 0, stream, residual, (const T*)delta,     \
+                                    (const T*)delta2, alpha, weight, bias, rows, (T*)out, n_out, hidden)))
+  if (wide) { MS_DYNAMIC_TANH(8); } else { MS_DYNAMIC_TANH(1); }
+#undef MS_DYNAMIC_TANH
+  MS_CHECK_LAUNCH("add_dynamic_tanh");
   return 0;
 }
 

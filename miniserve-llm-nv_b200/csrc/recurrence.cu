@@ -10,7 +10,9 @@
 //                               delta:  S = decay S, u = beta (v - S^T k), S = S + k u^T, y = S^T q
 //                               decay:  S = decay_h S + k v^T with a constant per head, y = S^T q (q, k, v through SiLU if asked)
 //                               channel delta: the delta form with one decay per head and key channel (rows of S)
-//   ms_low_rank_expand        the second product of a two-step (low-rank) projection, as it is, or turned into decays
+//                               channel decay: S = diag(decay) S + k v^T with one decay per token, head and key channel, y = S^T q
+//   ms_low_rank_expand        the second product of a two-step (low-rank) projection, as it is, or turned into decays of one
+//                             of two forms
 //   ms_head_norm_gate         y / bottom, divided by its root mean square per head, times a weight, times sigmoid or SiLU of a gate
 //   ms_gated_recurrence_scan  S = a S + sqrt(1 - a^2) i u per channel with a = exp(rate sigmoid(.)), times gelu_tanh of a branch
 //
@@ -110,7 +112,7 @@ __global__ void decay_gates_kernel(const float* __restrict__ logits, const float
 // way from memory into registers (kScanFetch keys, queries and values a thread: a chunk holds at most 256 kScanFetch of
 // each), so that the walk waits for memory once a request and not once a chunk.
 constexpr int kScanThreads = 256, kScanShift = 8;
-constexpr int kModeMemory = 0, kModeDelta = 1, kModeDecay = 2, kModeChannelDelta = 3;
+constexpr int kModeMemory = 0, kModeDelta = 1, kModeDecay = 2, kModeChannelDelta = 3, kModeChannelDecay = 4;
 constexpr int kPiecePad = 4;
 constexpr int kScanFetch = 8;
 
@@ -136,9 +138,10 @@ matrix_scan_kernel(const T* __restrict__ q, int q_ld, int q_col, const T* __rest
   grid_dependency_launch();
   extern __shared__ __align__(16) float matrix_smem[];
   // numbers of `gates` a token and head has: (keep, write, floor), (decay, beta), none (the decay is the head's constant:
-  // gates [heads]), or one logit whose sigmoid is beta (gates: rows of gate_ld numbers, the heads' logits from gate_col)
-  constexpr int G = MODE == kModeMemory ? 3 : MODE == kModeDelta ? 2 : MODE == kModeDecay ? 0 : 1;
-  constexpr bool CHANNEL = MODE == kModeChannelDelta;
+  // gates [heads]; or the decays are the channels'), or one logit whose sigmoid is beta (gates: rows of gate_ld numbers, the heads'
+  // logits from gate_col)
+  constexpr int G = MODE == kModeMemory ? 3 : MODE == kModeDelta ? 2 : MODE == kModeChannelDelta ? 1 : 0;
+  constexpr bool CHANNEL = MODE == kModeChannelDelta || MODE == kModeChannelDecay;
   constexpr int PIECE = R + kPiecePad;
   const int LPC = 1 << lpc_shift, cols_per_block = kScanThreads >> lpc_shift;
   const int row = LPC * PIECE;                                // floats of a token's key (or query) in shared memory
@@ -154,7 +157,7 @@ matrix_scan_kernel(const T* __restrict__ q, int q_ld, int q_col, const T* __rest
   float* qs = ks + tok * row;                                 // [tok][row]
   float* vs = qs + tok * row;                                 // [tok][cols_per_block]
   float* gs = vs + tok * cols_per_block;                      // [tok][4]
-  float* ds = gs + tok * 4;                                   // [tok][row]: the key channels' decays (channel delta only)
+  float* ds = gs + tok * 4;                                   // [tok][row]: the key channels' decays (channel forms only)
   const float head_decay = MODE == kModeDecay ? gates[head] : 1.f;
   float* kept = states + (long long)state_slots[request] * state_stride + state_offset + ((size_t)head * columns + (active ? col : 0)) * dim;
   float s[R];
@@ -205,7 +208,7 @@ matrix_scan_kernel(const T* __restrict__ q, int q_ld, int q_col, const T* __rest
       const int idx = tid + kScanThreads * j, tt = idx >> col_shift, c = idx & (cols_per_block - 1);
       next_v[j] = (tt < len && c < cols_here) ? v_head[(first + tt) * v_ld + c] : from_float<T>(1.f);      // (the column n)
     }
-    if (CHANNEL) {
+    if (MODE == kModeChannelDelta) {
       if (tid < len) next_g = sigmoid_f(gates[(first + tid) * gate_ld + gate_col + head]);
     } else if (G > 0) {
       if (tid < len * G) next_g = gates[((first + tid / (G > 0 ? G : 1)) * heads + head) * G + tid % (G > 0 ? G : 1)];
@@ -236,7 +239,7 @@ matrix_scan_kernel(const T* __restrict__ q, int q_ld, int q_col, const T* __rest
         vs[idx] = value;
       }
     }
-    if (CHANNEL) {
+    if (MODE == kModeChannelDelta) {
       if (tid < len) gs[tid * 4 + 1] = next_g;
     } else if (G > 0) {
       if (tid < len * G) gs[(tid / (G > 0 ? G : 1)) * 4 + tid % (G > 0 ? G : 1)] = next_g;
@@ -259,6 +262,20 @@ matrix_scan_kernel(const T* __restrict__ q, int q_ld, int q_col, const T* __rest
           s[r + 1] = keep * s[r + 1] + write * kv.y;
           s[r + 2] = keep * s[r + 2] + write * kv.z;
           s[r + 3] = keep * s[r + 3] + write * kv.w;
+          acc[0] += s[r] * qv.x;
+          acc[1] += s[r + 1] * qv.y;
+          acc[2] += s[r + 2] * qv.z;
+          acc[3] += s[r + 3] * qv.w;
+        }
+      } else if (MODE == kModeChannelDecay) {
+        const float4* dd = reinterpret_cast<const float4*>(ds + tt * row + sub * PIECE);
+#pragma unroll
+        for (int r = 0; r < R; r += 4) {
+          const float4 kv = kk[r >> 2], qv = qq[r >> 2], dv = dd[r >> 2];
+          s[r] = dv.x * s[r] + value * kv.x;
+          s[r + 1] = dv.y * s[r + 1] + value * kv.y;
+          s[r + 2] = dv.z * s[r + 2] + value * kv.z;
+          s[r + 3] = dv.w * s[r + 3] + value * kv.w;
           acc[0] += s[r] * qv.x;
           acc[1] += s[r + 1] * qv.y;
           acc[2] += s[r + 2] * qv.z;
@@ -322,11 +339,12 @@ matrix_scan_kernel(const T* __restrict__ q, int q_ld, int q_col, const T* __rest
 
 // The second product of a projection made in two steps through `rank` numbers: value[n, r] = sum_j mid[n, col + j] w[r, j]
 // with mid float32 (rows of ld numbers) and w float32 [rows, rank].  decay == 0: out[n, r] = value in the type T.
-// decay != 0 (T float): out[n, r] = exp(-exp(a_log[r / per_head]) softplus(value + bias[r])), a decay per head and channel.
+// decay == 1 (T float): out[n, r] = exp(-exp(a_log[r / per_head]) softplus(value + bias[r])), a decay per head and channel.
+// decay == 2 (T float): out[n, r] = sigmoid(value + bias[r])^inv_tau, formed as exp(inv_tau log sigmoid).
 template <typename T>
 __global__ void low_rank_expand_kernel(const float* __restrict__ mid, int ld, int col, int rank, const float* __restrict__ w,
                                        int rows, int decay, const float* __restrict__ a_log, const float* __restrict__ bias,
-                                       int per_head, T* __restrict__ out, long long total) {
+                                       int per_head, float inv_tau, T* __restrict__ out, long long total) {
   grid_dependency_wait();
   grid_dependency_launch();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -340,7 +358,8 @@ __global__ void low_rank_expand_kernel(const float* __restrict__ mid, int ld, in
     const float* wr = w + (size_t)r * rank;
     for (int j = 0; j < rank; ++j) sum += row[j] * wr[j];
   }
-  if (decay) sum = expf(-expf(a_log[r / per_head]) * softplus_f(sum + bias[r]));
+  if (decay == 1) sum = expf(-expf(a_log[r / per_head]) * softplus_f(sum + bias[r]));
+  else if (decay == 2) sum = expf(inv_tau * log_sigmoid_f(sum + bias[r]));
   out[i] = from_float<T>(sum);
 }
 
@@ -354,7 +373,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 low_rank_expand_tiled_kernel(const float* __restrict__ mid, int ld, int col, int rank, const float* __restrict__ wt, int rows,
                              int decay, const float* __restrict__ a_log, const float* __restrict__ bias, int per_head,
-                             T* __restrict__ out, int n_tokens) {
+                             float inv_tau, T* __restrict__ out, int n_tokens) {
   grid_dependency_wait();
   grid_dependency_launch();
   extern __shared__ float expand_smem[];                      // [kExpandTokens][rank]
@@ -376,10 +395,13 @@ low_rank_expand_tiled_kernel(const float* __restrict__ mid, int ld, int col, int
     for (int t = 0; t < kExpandTokens; ++t) acc[t] += expand_smem[t * rank + j] * w;
   }
   float rate = 0.f, b = 0.f;
-  if (decay) rate = -expf(a_log[r / per_head]), b = bias[r];
+  if (decay) b = bias[r];
+  if (decay == 1) rate = -expf(a_log[r / per_head]);
 #pragma unroll
   for (int t = 0; t < kExpandTokens; ++t) {
-    if (t < len) out[(size_t)(t0 + t) * rows + r] = from_float<T>(decay ? expf(rate * softplus_f(acc[t] + b)) : acc[t]);
+    if (t >= len) break;
+    const float value = decay == 1 ? expf(rate * softplus_f(acc[t] + b)) : decay == 2 ? expf(inv_tau * log_sigmoid_f(acc[t] + b)) : acc[t];
+    out[(size_t)(t0 + t) * rows + r] = from_float<T>(value);
   }
 }
 
@@ -624,7 +646,7 @@ static int scan_sm_count() {
 // numbers of type `dtype`; y float32 [tokens, heads, vdim].  max_query_len: an upper bound of the tokens a request brings.
 // mode 2 (decay): gates [heads], the heads' constant decays; state [heads, vdim, dim].  mode 3 (channel delta): gates are rows
 // of gate_ld float32 numbers whose columns gate_col .. gate_col + heads hold the logits of beta; channel_decay float32
-// [tokens, heads, dim]; state [heads, vdim, dim].  input_act != 0: q, k and v pass SiLU as they are read.
+// [tokens, heads, dim]; state [heads, vdim, dim].  mode 4 (channel decay): channel_decay as in mode 3, gates unused; the same state.  input_act != 0: q, k and v pass SiLU as they are read.
 MS_EXPORT int ms_matrix_scan(int mode, const void* q, int q_ld, int q_col, const void* k, int k_ld, int k_col, const void* v,
                              int v_ld, int v_col, int dtype, float q_scale, const float* gates, float* states,
                              long long state_stride, int state_offset, const int* state_slots, const int* query_start,
@@ -632,7 +654,8 @@ MS_EXPORT int ms_matrix_scan(int mode, const void* q, int q_ld, int q_col, const
                              float* bottom, int gate_ld, int gate_col, const float* channel_decay, int input_act,
                              cudaStream_t stream) {
   if (n_requests == 0 || max_query_len <= 0 || heads == 0) return 0;
-  MS_REQUIRE(mode >= kModeMemory && mode <= kModeChannelDelta, "matrix_scan: mode %d", mode);
+  MS_REQUIRE(mode >= kModeMemory && mode <= kModeChannelDecay, "matrix_scan: mode %d", mode);
+  MS_REQUIRE(mode != kModeChannelDecay || channel_decay != nullptr, "matrix_scan: the channel form needs the channels' decays");
   MS_REQUIRE(mode != kModeChannelDelta || (channel_decay != nullptr && gate_col >= 0 && gate_col + heads <= gate_ld),
              "matrix_scan: the channel form needs the channels' decays and the heads' logits (columns %d.. of %d)", gate_col, gate_ld);
   MS_REQUIRE(kv_heads > 0 && heads % kv_heads == 0 && dim >= 1 && dim <= 512 && vdim >= 1, "matrix_scan: %d/%d heads of %d/%d",
@@ -661,7 +684,7 @@ MS_EXPORT int ms_matrix_scan(int mode, const void* q, int q_ld, int q_col, const
   const int r = piece(lpc_shift);
   const int cols_per_block = kScanThreads >> lpc_shift;
   const int columns = mode == kModeMemory ? vdim + 1 : vdim;
-  const int row_floats = (mode == kModeChannelDelta ? 3 : 2) * ((r + kPiecePad) << lpc_shift) + cols_per_block + 4;
+  const int row_floats = (mode >= kModeChannelDelta ? 3 : 2) * ((r + kPiecePad) << lpc_shift) + cols_per_block + 4;
   // a chunk: at most 16 tokens, kScanThreads kScanFetch keys and as many values (what the threads hold of the next chunk)
   // and 40 KB of shared memory
   int tok = max_query_len < 16 ? max_query_len : 16;
@@ -685,6 +708,9 @@ MS_EXPORT int ms_matrix_scan(int mode, const void* q, int q_ld, int q_col, const
   } else if (mode == kModeChannelDelta) {
     if (r == 4) { MS_MATRIX_SCAN(4, kModeChannelDelta); } else if (r == 8) { MS_MATRIX_SCAN(8, kModeChannelDelta); }
     else if (r == 16) { MS_MATRIX_SCAN(16, kModeChannelDelta); } else { MS_MATRIX_SCAN(32, kModeChannelDelta); }
+  } else if (mode == kModeChannelDecay) {
+    if (r == 4) { MS_MATRIX_SCAN(4, kModeChannelDecay); } else if (r == 8) { MS_MATRIX_SCAN(8, kModeChannelDecay); }
+    else if (r == 16) { MS_MATRIX_SCAN(16, kModeChannelDecay); } else { MS_MATRIX_SCAN(32, kModeChannelDecay); }
   } else {
     if (r == 4) { MS_MATRIX_SCAN(4, kModeDelta); } else if (r == 8) { MS_MATRIX_SCAN(8, kModeDelta); }
     else if (r == 16) { MS_MATRIX_SCAN(16, kModeDelta); } else { MS_MATRIX_SCAN(32, kModeDelta); }
@@ -695,17 +721,19 @@ MS_EXPORT int ms_matrix_scan(int mode, const void* q, int q_ld, int q_col, const
 }
 
 // mid float32 rows of ld numbers (the first product's results from column col); wt float32 [rank, rows], the second matrix
-// TRANSPOSED; out [tokens, rows] of type `dtype`, or, decay != 0, float32 decays exp(-exp(a_log[row / per_head]) softplus(. +
-// bias[row])).  wt null (rank == rows): the numbers of mid themselves take the place of the product.
+// TRANSPOSED; out [tokens, rows] of type `dtype`, or float32 decays: decay 1, exp(-exp(a_log[row / per_head]) softplus(. +
+// bias[row])), decay 2, sigmoid(. + bias[row])^inv_tau.  wt null (rank == rows): the numbers of mid themselves take the place of the product.
 MS_EXPORT int ms_low_rank_expand(const float* mid, int ld, int col, int rank, const float* wt, int rows, int decay,
-                                 const float* a_log, const float* bias, int per_head, void* out, int dtype, int n_tokens,
-                                 cudaStream_t stream) {
+                                 const float* a_log, const float* bias, int per_head, float inv_tau, void* out, int dtype,
+                                 int n_tokens, cudaStream_t stream) {
   const long long total = (long long)n_tokens * rows;
   if (total == 0) return 0;
   MS_REQUIRE(rank >= 1 && col >= 0 && col + rank <= ld, "low_rank_expand: %d numbers from column %d of rows of %d", rank, col, ld);
   MS_REQUIRE(wt != nullptr || rank == rows, "low_rank_expand: without a second matrix the %d numbers are the %d results", rank, rows);
-  MS_REQUIRE(!decay || (a_log && bias && per_head >= 1 && rows % per_head == 0 && dtype == MS_F32),
+  MS_REQUIRE(decay >= 0 && decay <= 2, "low_rank_expand: decay form %d", decay);
+  MS_REQUIRE(decay != 1 || (a_log && bias && per_head >= 1 && rows % per_head == 0 && dtype == MS_F32),
              "low_rank_expand: decays are float32 and need A_log, a bias and the heads' size (%d rows, %d a head)", rows, per_head);
+  MS_REQUIRE(decay != 2 || (bias && inv_tau > 0.f && dtype == MS_F32), "low_rank_expand: decays are float32 and need a bias and a power (%f)", inv_tau);
   if (wt != nullptr) {
     const size_t smem = (size_t)kExpandTokens * rank * sizeof(float);
     MS_REQUIRE(smem <= 48 * 1024, "low_rank_expand: %d numbers a token do not fit the shared memory", rank);
@@ -713,14 +741,14 @@ MS_EXPORT int ms_low_rank_expand(const float* mid, int ld, int col, int rank, co
     MS_REQUIRE(token_tiles <= 65535, "low_rank_expand: %d tokens in one launch is too many", n_tokens);
     dim3 grid((rows + 255) / 256, token_tiles);
     MS_REC_DISPATCH(dtype, (ms::launch(low_rank_expand_tiled_kernel<T>, grid, 256, smem, stream, mid, ld, col, rank, wt, rows, decay,
-                                       a_log, bias, per_head, (T*)out, n_tokens)));
+                                       a_log, bias, per_head, inv_tau, (T*)out, n_tokens)));
     MS_CHECK_LAUNCH("low_rank_expand");
     return 0;
   }
   const long long blocks = (total + 255) / 256;
   MS_REQUIRE(blocks < 2147483647LL, "low_rank_expand: %lld numbers in one launch is too many", total);
   MS_REC_DISPATCH(dtype, (ms::launch(low_rank_expand_kernel<T>, (unsigned)blocks, 256, 0, stream, mid, ld, col, rank, wt, rows, decay,
-                                     a_log, bias, per_head, (T*)out, total)));
+                                     a_log, bias, per_head, inv_tau, (T*)out, total)));
   MS_CHECK_LAUNCH("low_rank_expand");
   return 0;
 }

@@ -49,9 +49,17 @@ __device__ __forceinline__ float clamped_times(float gate, float up, float limit
   return g * (g >= 0.f ? r : e * r) * (u + 1.f);
 }
 
-// A gated activation: silu(g) u, or the clamped one where a limit (above 0) is given.
-__device__ __forceinline__ float gated_times(float g, float u, float limit) {
-  return limit > 0.f ? clamped_times(g, u, limit) : silu_times(g, u);
+// gelu_tanh(g) u
+__device__ __forceinline__ float gelu_times(float g, float u) {
+  const float y = gelu_tanh_exponent(g);
+  const float e = __expf(-fabsf(y));
+  const float r = __fdividef(1.0f, 1.0f + e);
+  return g * (y >= 0.f ? r : e * r) * u;
+}
+
+// A gated activation by its code.
+__device__ __forceinline__ float gated_times(float g, float u, int activation, float limit) {
+  return activation == kGateClamped ? clamped_times(g, u, limit) : activation == kGateGelu ? gelu_times(g, u) : silu_times(g, u);
 }
 
 // Barriers of the computing warps alone (the copying warp takes no part).

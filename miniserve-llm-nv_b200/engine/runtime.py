@@ -138,7 +138,7 @@ def _report_attention_kernels(model: DecoderModel, dtype: torch.dtype, page_size
         if not isinstance(need, PagedKVNeed):
             continue
         n_q = getattr(mixer, "attention_heads", None) or getattr(mixer, "num_heads", need.num_kv_heads)
-        modified = bool(getattr(mixer, "score_softcap", None)) or getattr(mixer, "score_bias_slopes", None) is not None
+        modified = getattr(mixer, "score_bias_slopes", None) is not None
         names = kernels.attention_kernels(dtype, need.head_dim, n_q, need.num_kv_heads, page_size, modified, need.value_dim,
                                           bool(getattr(mixer, "general", False)), need.chunk, need.num_value_heads != need.num_kv_heads)
         chosen.append(dict(group=plan.group, head_dim=need.head_dim, window=need.window, **names))
@@ -147,5 +147,5 @@ def _report_attention_kernels(model: DecoderModel, dtype: torch.dtype, page_size
                 "cache group %d (head size %d, %d/%d heads, pages of %d%s): decode steps on the %s kernel, prompt "
                 "portions on the %s kernel%s", plan.group, need.head_dim, n_q, need.num_kv_heads, page_size,
                 f", window {need.window}" if need.window else "", names["decode"], names["prompt"],
-                " (no tensor-core kernel is built for this head size or for modified scores)" if slow else "")
+                " (no tensor-core kernel is built for this head size or for a bias of the scores)" if slow else "")
     return chosen

@@ -16,7 +16,7 @@ import torch
 
 from . import build
 
-ABI_VERSION = 12
+ABI_VERSION = 13
 log = logging.getLogger("miniserve_b200")
 _library: Optional[ctypes.CDLL] = None
 
@@ -215,6 +215,28 @@ def add_layernorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight:
         _ptr(bias2), _i(_code(weight.dtype)), _f(eps), _ptr(rows), _ptr(out), _ptr(out2), _i(n_out), _i(hidden), _stream()))
 
 
+def add_dynamic_tanh(residual: torch.Tensor, delta: Optional[torch.Tensor], alpha: float, weight: torch.Tensor, bias: torch.Tensor,
+                     out: torch.Tensor, rows: Optional[torch.Tensor] = None, delta2: Optional[torch.Tensor] = None) -> None:
+    """Adds ``delta`` (or ``delta + delta2``, summed in float32) into the float32 ``residual`` (in place) and writes ``weight * tanh(alpha
+    * x) + bias`` of the sum to ``out``, entry by entry (weight and bias float32 ``[H]``).  With ``rows`` (int32 ``[K]``) only those
+    rows are written, to ``out [K, H]``, and the residual is left untouched."""
+    hidden = residual.shape[1]
+    n_out = residual.shape[0] if rows is None else rows.numel()
+    _want(residual, "residual", torch.float32)
+    _want(out, "out", None, (n_out, hidden))
+    _want(weight, "weight", torch.float32, (hidden,))
+    _want(bias, "bias", torch.float32, (hidden,))
+    if delta is None and delta2 is not None:
+        delta, delta2 = delta2, None
+    for name, tensor in (("delta", delta), ("delta2", delta2)):
+        if tensor is not None:
+            _want(tensor, name, out.dtype, residual.shape)
+    if rows is not None:
+        _want(rows, "rows", torch.int32)
+    _check(library().ms_add_dynamic_tanh(_ptr(residual), _ptr(delta), _ptr(delta2), _i(_code(out.dtype)), _f(alpha), _ptr(weight),
+                                         _ptr(bias), _ptr(rows), _ptr(out), _i(n_out), _i(hidden), _stream()))
+
+
 def stream_to_columns(residual: torch.Tensor, delta: Optional[torch.Tensor], out: torch.Tensor, col: int,
                       delta2: Optional[torch.Tensor] = None) -> None:
     """``out[n, col : col + H] = residual[n] + (delta[n] + delta2[n])`` rounded once to ``out``'s type: the stream with what is
@@ -235,7 +257,8 @@ def qkv_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, n_q: int
                 slots: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
                 cos_sin: Optional[torch.Tensor], rotary_dim: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
                 q_out: torch.Tensor, interleaved: bool = False, bias: Optional[torch.Tensor] = None,
-                value_heads: Optional[int] = None) -> None:
+                value_heads: Optional[int] = None, kept_values: Optional[torch.Tensor] = None,
+                mix_share: Optional[float] = None) -> None:
     """Per-head RMSNorm of q and k, rotation of their first ``rotary_dim`` entries (entry i with entry i + rotary_dim / 2,
     or, ``interleaved``, entry 2i with entry 2i + 1), and the append of k and v
     to one layer's pools, for a projection ``proj [N, ld]`` whose columns are laid out freely: query head h at
@@ -245,13 +268,19 @@ def qkv_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, n_q: int
     norm weights float32 ``[head_dim]`` or None; ``cos_sin`` float32 ``[N, rotary_dim / 2, 2]`` or None.  ``bias`` (float32
     ``[ld]``, column by column as ``proj``): the projection's bias, added in float32 as the heads are read.  ``value_heads``
     (a divisor of ``n_kv``; None: ``n_kv``): the projection and the value pool ``[pages, value_heads, page_size, value_dim]`` hold
-    that many value heads (key heads that share values: key head g reads value head ``g % value_heads``)."""
+    that many value heads (key heads that share values: key head g reads value head ``g % value_heads``).  ``kept_values [N,
+    value_heads * value_dim]``: without ``mix_share`` it receives the tokens' values (biases included); with it the values become
+    ``(1 - mix_share) v + mix_share kept_values`` in float32 before they are stored."""
     n, ld = proj.shape
     value_heads = n_kv if value_heads is None else int(value_heads)
     if value_heads < 1 or n_kv % value_heads:
         raise KernelError(f"qkv_prepare: {value_heads} value heads for {n_kv} key heads")
     if bias is not None:
         _want(bias, "bias", torch.float32, (ld,))
+    if kept_values is not None:
+        _want(kept_values, "kept_values", proj.dtype, (n, value_heads * value_dim))
+    elif mix_share is not None:
+        raise KernelError("qkv_prepare: a share without the values to mix in")
     _want(proj, "proj")
     _want(q_out, "q_out", proj.dtype, (n, n_q, head_dim))
     own = k_col >= 0
@@ -276,7 +305,8 @@ def qkv_prepare(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, n_q: int
         _ptr(proj), _i(_code(proj.dtype)), _i(ld), _i(q_col), _i(k_col if own else -1), _i(v_col if own else -1), _i(n_q), _i(n_kv),
         _i(head_dim), _i(value_dim), _ptr(slots) if own else None, _ptr(q_weight), _ptr(k_weight) if own else None, _f(eps),
         _ptr(cos_sin), _i(rotary_dim), _ptr(k_pool) if own else None, _ptr(v_pool) if own else None,
-        _i(k_pool.shape[2]) if own else 1, _ptr(q_out), _i(n), _i(1 if interleaved else 0), _ptr(bias), _i(value_heads), _stream()))
+        _i(k_pool.shape[2]) if own else 1, _ptr(q_out), _i(n), _i(1 if interleaved else 0), _ptr(bias), _i(value_heads),
+        _ptr(kept_values), _i(0 if mix_share is None else 1), _f(mix_share or 0.0), _stream()))
 
 
 def qkv_prepare_rows(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, n_q: int, n_kv: int, head_dim: int, value_dim: int,
@@ -362,11 +392,24 @@ def qk_norm_rope_append(qkv: torch.Tensor, slots: torch.Tensor, q_weight: Option
         _i(n_q), _i(n_kv), _i(head_dim), _ptr(q_out), _i(n), _stream()))
 
 
+GATE_ACTIVATIONS = {"silu": 0, "clamped_glu": 1, "gelu_tanh": 2}
+
+
+def _gate_code(activation: str, limit: Optional[float]) -> int:
+    """The code of a gated activation; a limit alone says ``clamped_glu``."""
+    if limit and activation in ("silu", "clamped_glu"):
+        return GATE_ACTIVATIONS["clamped_glu"]
+    if activation not in GATE_ACTIVATIONS or activation == "clamped_glu" or limit:
+        raise KernelError(f"gated activation {activation!r} with limit {limit}")
+    return GATE_ACTIVATIONS[activation]
+
+
 def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, paired: bool = False, bias: Optional[torch.Tensor] = None,
-             limit: Optional[float] = None) -> None:
+             limit: Optional[float] = None, activation: str = "silu") -> None:
     """``out[n, c] = silu(gate_up[n, c]) * gate_up[n, I + c]`` for gate_up ``[N, 2 I]``.  With ``bias`` (float32 ``[2 I]``,
     not with ``paired``) it is added to both halves first, in float32.  ``limit`` (not with ``bias``): the clamped gated
     activation instead, ``g sigmoid(1.702 g) (u + 1)`` with ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``.
+    ``activation="gelu_tanh"`` (not with ``bias``): the tanh form of GELU in place of SiLU.
 
     ``paired``: the columns come as :func:`interleave_gate_up` orders a weight's rows (eight gate columns, then
     the up columns of the same features, and so on): ``out[n, 8 j + r] = silu(gate_up[n, 16 j + r]) *
@@ -377,12 +420,12 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, paired: bool = False, bia
     _want(out, "out", gate_up.dtype)
     if bias is not None:
         _want(bias, "bias", torch.float32, (2 * inter,))
-        if paired or limit:
+        if paired or _gate_code(activation, limit):
             raise KernelError("silu_mul: a bias goes with the plain layout (gate columns, then up columns) and the plain activation")
         _check(library().ms_silu_mul_bias(_ptr(gate_up), _i(_code(gate_up.dtype)), _ptr(bias), _ptr(out), _i(n), _i(inter), _stream()))
         return
     _check(library().ms_silu_mul(_ptr(gate_up), _i(_code(gate_up.dtype)), _ptr(out), _i(n), _i(inter),
-                                 _i(1 if paired else 0), _f(limit or 0.0), _stream()))
+                                 _i(1 if paired else 0), _i(_gate_code(activation, limit)), _f(limit or 0.0), _stream()))
 
 
 def add_bias(x: torch.Tensor, bias: torch.Tensor) -> None:
@@ -501,7 +544,7 @@ def attention_kernels(dtype: torch.dtype, head_dim: int, n_q: int, n_kv: int, pa
     """Which kernel :func:`paged_attention` runs for these sizes: ``{"decode": name, "prompt": name}`` with the
     names ``tcgen05``, ``mma.sync`` and ``general`` (float32 arithmetic, any size; the only one of the float32
     path, and what bfloat16 falls back to for head sizes the tensor-core kernels are not built for and for
-    scores with a soft cap or a distance bias)."""
+    ``modified_scores``, a distance bias)."""
     lib = library()
     value_dim = head_dim if value_dim is None else value_dim
     chunk = chunk or (1 if shared_values else None)      # (key heads that share value heads: the same two kernels)
@@ -544,8 +587,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
 
     Score modifiers, both off by default: ``softcap`` turns a scaled score ``s`` into ``softcap * tanh(s /
     softcap)``; ``bias_slopes`` (float32 ``[n_q]``) adds ``slope[head] * (key position - query position)``
-    after it.  The general kernel implements them; the tensor-core kernels do not, so a call with either
-    runs the general kernel whatever the sizes.
+    after it.  Every kernel implements the soft cap; the bias runs the general kernel whatever the sizes.
 
     bfloat16 with a head size the tensor-core kernels are built for runs there
     (``max_query_len``/``max_context_len`` are upper bounds used to shape their grids); everything
@@ -583,7 +625,8 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     if isinstance(sink, torch.Tensor):
         _want(sink, "sink", torch.float32, (n_q,))
         sink, sink_scores = True, sink
-    modified = bool(softcap) or bias_slopes is not None
+    modified = bias_slopes is not None
+    cap = _f(softcap if softcap else 0.0)
     if bias_slopes is not None:
         _want(bias_slopes, "bias_slopes", torch.float32, (n_q,))
     # the general form (a sink, a gate, value heads of their own size) at sizes the unrolled tensor-core kernels are not built
@@ -606,7 +649,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                 _ptr(query_start[first:last + 1]), _ptr(context_lens[first:last]), _i(k_pool.shape[2]), _i(n_q), _i(n_kv),
                 _i(head_dim), _i(value_dim), _f(scale), _i(window if window else 0), _ptr(out), _ptr(part_o), _ptr(part_lse),
                 _i(splits), _i(count), _i(longest), _i(rows), _i(1 if sink else 0), _ptr(sink_scores), gate_ptr, _i(gate_ld), _i(first_row),
-                _i(chunk or 0), _i(n_v), _stream()))
+                _i(chunk or 0), _i(n_v), cap, _stream()))
 
         single = 0
         if host_query_start and max_query_len > 1 and len(host_query_start) == n_requests + 1:
@@ -623,7 +666,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
         _check(lib.ms_paged_attention_generic(
             _ptr(q), _i(_code(q.dtype)), _ptr(k_pool), _ptr(v_pool), _ptr(block_tables), _i(block_tables.shape[1]),
             _ptr(request_of_token), _ptr(positions), _i(k_pool.shape[2]), _i(n_q), _i(n_kv), _i(head_dim),
-            _f(scale), _i(window if window else 0), _f(softcap if softcap else 0.0), _ptr(bias_slopes), _ptr(out),
+            _f(scale), _i(window if window else 0), cap, _ptr(bias_slopes), _ptr(out),
             _i(n), _i(value_dim), _i(1 if sink else 0), _ptr(sink_scores), gate_ptr, _i(gate_ld), _i(chunk or 0), _i(n_v), _stream()))
         return
 
@@ -635,7 +678,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
         tables, starts, lens = block_tables[first:last], query_start[first:last + 1], context_lens[first:last]
         count = last - first
         group = n_q // n_kv
-        if (USE_TCGEN05_ATTENTION and longest * group > 16 and (ATTENTION_IN_TURNS or not (sink or gate is not None))
+        if (USE_TCGEN05_ATTENTION and longest * group > 16 and (ATTENTION_IN_TURNS or not (sink or gate is not None or softcap))
                 and lib.ms_attention_tcgen05_supports(_i(head_dim), _i(n_q), _i(n_kv), _i(k_pool.shape[2]))):
             # prompt portions: the TMA + tcgen05 + tensor-memory kernel, its softmax groups taking the key tiles in
             # turn (that form also takes the sink and the gate) or working on each together
@@ -644,7 +687,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                     _ptr(q), _ptr(k_pool), _ptr(v_pool), _i(k_pool.shape[0]), _ptr(tables), _i(block_tables.shape[1]),
                     _ptr(starts), _ptr(lens), _i(k_pool.shape[2]), _i(n_q), _i(n_kv), _i(head_dim), _f(scale),
                     _i(window if window else 0), _ptr(out), _i(count), _i(longest), _i(n),
-                    _ptr(device_error_flag(q.device)), _i(1 if sink else 0), _ptr(sink_scores), gate_ptr, _i(gate_ld), _stream()))
+                    _ptr(device_error_flag(q.device)), _i(1 if sink else 0), _ptr(sink_scores), gate_ptr, _i(gate_ld), cap, _stream()))
                 return
             _check(lib.ms_paged_attention_tcgen05(
                 _ptr(q), _ptr(k_pool), _ptr(v_pool), _i(k_pool.shape[0]), _ptr(tables), _i(block_tables.shape[1]),
@@ -661,7 +704,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
             _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(tables), _i(block_tables.shape[1]), _ptr(starts), _ptr(lens),
             _i(k_pool.shape[2]), _i(n_q), _i(n_kv), _i(head_dim), _f(scale), _i(window if window else 0), _ptr(out),
             _ptr(part_o), _ptr(part_lse), _i(splits), _i(count), _i(longest), _i(rows), _i(1 if sink else 0), _ptr(sink_scores),
-            gate_ptr, _i(gate_ld), _i(first_row), _stream()))
+            gate_ptr, _i(gate_ld), _i(first_row), cap, _stream()))
 
     leading_single = 0
     if host_query_start and max_query_len > 1 and len(host_query_start) == n_requests + 1:
@@ -957,7 +1000,8 @@ def gated_group_norm(y: torch.Tensor, proj: torch.Tensor, z_col: int, weight: to
 # --------------------------------------------------------------------------- recurrences that carry a matrix or a vector
 
 MAX_MATRIX_SCAN_DIM = 512     # entries of a query or key that matrix_scan spreads over a column's lanes (16 lanes x 32)
-MATRIX_SCAN_MODES = {"memory": 0, "delta": 1, "decay": 2, "channel_delta": 3}
+MATRIX_SCAN_MODES = {"memory": 0, "delta": 1, "decay": 2, "channel_delta": 3, "channel_decay": 4}
+MAX_EXPAND_RANK = 1024        # numbers between the two products of low_rank_expand
 HEAD_GATE_ACTIVATIONS = {"sigmoid": 0, "silu": 1}
 
 
@@ -1014,7 +1058,7 @@ def decay_gates(logits: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor
 
 
 def matrix_scan(mode: str, q: torch.Tensor, q_col: int, k: torch.Tensor, k_col: int, v: torch.Tensor, v_col: int,
-                gates: torch.Tensor, states: torch.Tensor, state_offset: int, state_slots: torch.Tensor,
+                gates: Optional[torch.Tensor], states: torch.Tensor, state_offset: int, state_slots: torch.Tensor,
                 query_start: torch.Tensor, max_query_len: int, heads: int, kv_heads: int, dim: int, vdim: int, y: torch.Tensor,
                 q_scale: float = 1.0, bottom: Optional[torch.Tensor] = None, gate_col: int = 0,
                 channel_decay: Optional[torch.Tensor] = None, input_activation: str = "none") -> None:
@@ -1029,7 +1073,8 @@ def matrix_scan(mode: str, q: torch.Tensor, q_col: int, k: torch.Tensor, k_col: 
     The state holds ``[H, vdim, dim]``.  ``y`` float32 ``[N, H, vdim]``.
     ``"decay"``: ``gates [H]``, a constant decay per head; ``S = decay S + k v^T``, ``y = S^T q`` (a linear attention).
     ``"channel_delta"``: the delta form with a decay per head and key channel, ``channel_decay`` float32 ``[N, H * dim]``, acting on
-    the rows of ``S``; ``gates`` is float32 ``[N, ld]`` whose columns ``gate_col .. gate_col + H`` hold the logits of beta.  Both
+    the rows of ``S``; ``gates`` is float32 ``[N, ld]`` whose columns ``gate_col .. gate_col + H`` hold the logits of beta.
+    ``"channel_decay"``: ``S = diag(channel_decay) S + k v^T``, ``y = S^T q`` (a gated linear attention; ``gates`` None).  All three
     keep ``[H, vdim, dim]``.  ``input_activation="silu"``: q, k and v pass SiLU as they are read."""
     code = MATRIX_SCAN_MODES[mode]
     n = y.shape[0]
@@ -1049,6 +1094,8 @@ def matrix_scan(mode: str, q: torch.Tensor, q_col: int, k: torch.Tensor, k_col: 
         if gates.dim() != 2 or gates.shape[0] != n or gate_col < 0 or gate_col + heads > gates.shape[1]:
             raise KernelError(f"matrix_scan: the logits of beta from column {gate_col} of {tuple(gates.shape)} for {heads} heads")
         gate_ld = gates.shape[1]
+    elif code == 4:
+        _want(channel_decay, "channel_decay", torch.float32, (n, heads * dim))
     else:
         _want(gates, "gates", torch.float32, (n, heads, 3 if code == 0 else 2))
     _want(y, "y", torch.float32, (n, heads, vdim))
@@ -1063,7 +1110,7 @@ def matrix_scan(mode: str, q: torch.Tensor, q_col: int, k: torch.Tensor, k_col: 
                                     _i(v.shape[1]), _i(v_col), _i(_code(q.dtype)), _f(q_scale), _ptr(gates), _ptr(states), stride,
                                     _i(state_offset), _ptr(state_slots), _ptr(query_start), _i(n_requests), _i(max_query_len),
                                     _i(heads), _i(kv_heads), _i(dim), _i(vdim), _ptr(y), _ptr(bottom), _i(gate_ld), _i(gate_col),
-                                    _ptr(channel_decay) if code == 3 else None, _i(CONV_ACTIVATIONS[input_activation]), _stream()))
+                                    _ptr(channel_decay) if code >= 3 else None, _i(CONV_ACTIVATIONS[input_activation]), _stream()))
 
 
 def channel_decays(logits: torch.Tensor, col: int, a_log: torch.Tensor, dt_bias: torch.Tensor, per_head: int, out: torch.Tensor) -> None:
@@ -1076,27 +1123,31 @@ def channel_decays(logits: torch.Tensor, col: int, a_log: torch.Tensor, dt_bias:
     _want(a_log, "a_log", torch.float32, (rows // max(per_head, 1),))
     _want(dt_bias, "dt_bias", torch.float32, (rows,))
     _check(library().ms_low_rank_expand(_ptr(logits), _i(ld), _i(col), _i(rows), None, _i(rows), _i(1), _ptr(a_log), _ptr(dt_bias),
-                                        _i(per_head), _ptr(out), _i(0), _i(n), _stream()))
+                                        _i(per_head), _f(0.0), _ptr(out), _i(0), _i(n), _stream()))
 
 
 def low_rank_expand(mid: torch.Tensor, col: int, weight_t: torch.Tensor, out: torch.Tensor, a_log: Optional[torch.Tensor] = None,
-                    bias: Optional[torch.Tensor] = None, per_head: int = 0) -> None:
+                    bias: Optional[torch.Tensor] = None, per_head: int = 0, tau: Optional[float] = None) -> None:
     """The second product of a projection made in two steps: ``value[n, r] = sum_j mid[n, col + j] weight_t[j, r]`` with ``mid``
     float32 ``[N, ld]`` and ``weight_t`` float32 ``[rank, R]``, the second matrix TRANSPOSED (the kernel's threads then read
     consecutive numbers).  Without ``a_log``: ``out [N, R]`` (any type) receives the values.
     With ``a_log`` (float32 ``[R / per_head]``) and ``bias`` (float32 ``[R]``): ``out`` float32 receives the decays
-    ``exp(-exp(a_log[r // per_head]) softplus(value + bias[r]))``."""
+    ``exp(-exp(a_log[r // per_head]) softplus(value + bias[r]))``.
+    With ``tau`` and ``bias``: ``out`` float32 receives the decays ``sigmoid(value + bias[r])^(1 / tau)``."""
     n, ld = mid.shape
     rank, rows = weight_t.shape
     _want(mid, "mid", torch.float32)
     _want(weight_t, "weight_t", torch.float32)
-    decay = a_log is not None
-    if decay:
+    decay = 1 if a_log is not None else 2 if tau is not None else 0
+    if decay == 1:
         _want(a_log, "a_log", torch.float32, (rows // max(per_head, 1),))
+    if decay:
         _want(bias, "bias", torch.float32, (rows,))
+    if tau is not None and (decay == 1 or not tau > 0):
+        raise KernelError(f"low_rank_expand: tau {tau} must be positive and goes without a_log")
     _want(out, "out", torch.float32 if decay else None, (n, rows))
-    _check(library().ms_low_rank_expand(_ptr(mid), _i(ld), _i(col), _i(rank), _ptr(weight_t), _i(rows), _i(1 if decay else 0),
-                                        _ptr(a_log), _ptr(bias), _i(per_head), _ptr(out), _i(_code(out.dtype)), _i(n), _stream()))
+    _check(library().ms_low_rank_expand(_ptr(mid), _i(ld), _i(col), _i(rank), _ptr(weight_t), _i(rows), _i(decay),
+                                        _ptr(a_log), _ptr(bias), _i(per_head), _f(1.0 / tau if tau is not None else 0.0), _ptr(out), _i(_code(out.dtype)), _i(n), _stream()))
 
 
 def head_norm_gate(y: torch.Tensor, bottom: Optional[torch.Tensor], weight: torch.Tensor, gate: torch.Tensor, gate_col: int,
@@ -1153,9 +1204,13 @@ def gated_recurrence_scan(u: torch.Tensor, pre: torch.Tensor, gate_bias: torch.T
 # --------------------------------------------------------------------------- routed experts
 
 
+GROUP_SCORES = ("largest", "two_largest")
+
+
 def router_topk(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], top: int, ids: torch.Tensor,
                 weights: torch.Tensor, logits: Optional[torch.Tensor] = None, *, choose_from: Optional[int] = None,
-                scoring: str = "chosen_softmax", correction: Optional[torch.Tensor] = None, groups: tuple = (1, 1)) -> None:
+                scoring: str = "chosen_softmax", correction: Optional[torch.Tensor] = None, groups: tuple = (1, 1),
+                group_score: str = "largest", normalize: Optional[float] = None, weight_scale: float = 1.0) -> None:
     """Router of a mixture of experts: float32 logits ``x @ weight^T + bias`` (``weight`` float32 ``[E, width]``), the
     ``top`` experts with the largest logits into ``ids`` int32 ``[N, top]`` (ties: the lower index) and the softmax over
     those logits alone into ``weights`` float32 ``[N, top]``.  ``logits`` float32 ``[N, E]``: scratch that is left holding
@@ -1166,7 +1221,8 @@ def router_topk(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
     ``score + correction`` (float32 ``[choose_from]`` or None) among the members of the ``groups[1]`` best of
     ``groups[0]`` equal groups of neighbours (a group's score: its largest choice score), and ``weights`` are the chosen
     outputs' scores as they are.  ``scoring="sigmoid"``: the same with ``sigmoid(logit)`` of every output on its own as its
-    score."""
+    score.  For both: ``group_score="two_largest"`` ranks a group by the sum of its two largest choice scores, ``normalize``
+    divides the weights by their sum plus that number, ``weight_scale`` multiplies them (afterwards)."""
     n, width = x.shape
     experts = weight.shape[0]
     if scoring in ("all_softmax", "sigmoid"):
@@ -1184,9 +1240,11 @@ def router_topk(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
         _want(weights, "weights", torch.float32, (n, top))
         _check(library().ms_router_choose(_ptr(x), _i(_code(x.dtype)), _ptr(weight), _ptr(bias), _i(width), _i(experts), _i(total),
                                           _i(top), _ptr(correction), _i(groups[0]), _i(groups[1]), _ptr(logits), _ptr(ids),
-                                          _ptr(weights), _i(n), _i(1 if scoring == "sigmoid" else 0), _stream()))
+                                          _ptr(weights), _i(n), _i(1 if scoring == "sigmoid" else 0), _i(GROUP_SCORES.index(group_score)),
+                                          _f(-1.0 if normalize is None else normalize), _f(weight_scale), _stream()))
         return
-    if scoring != "chosen_softmax" or correction is not None or tuple(groups) != (1, 1) or choose_from not in (None, experts):
+    if (scoring != "chosen_softmax" or correction is not None or tuple(groups) != (1, 1) or choose_from not in (None, experts)
+            or normalize is not None or weight_scale != 1.0):
         raise KernelError("router_topk: a correction, groups and rows that ride along need scoring='all_softmax'")
     if logits is None:
         logits = torch.empty((n, experts), dtype=torch.float32, device=x.device)
@@ -1532,11 +1590,12 @@ PAIR_WIDE = __import__("os").environ.get("MINISERVE_B200_PAIR_WIDE", "0") == "1"
 
 
 def linear_pair(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, add: bool = False, gated: bool = False,
-                row_stats: Optional["RowStats"] = None, wide: Optional[bool] = None, limit: Optional[float] = None) -> None:
+                row_stats: Optional["RowStats"] = None, wide: Optional[bool] = None, limit: Optional[float] = None,
+                activation: str = "silu") -> None:
     """``out = x @ weight^T`` by the kernel in which two thread blocks share each 256 x 256 tile (tcgen05 with
     ``cta_group::2``).  ``add``: ``out += ...`` on a float32 ``out``.  ``gated``: ``weight`` is
-    :func:`interleave_gate_up` of a gate and an up projection and ``out [M, N / 2] = silu(gate) * up`` (``limit``: the
-    clamped activation of :func:`silu_mul`).
+    :func:`interleave_gate_up` of a gate and an up projection and ``out [M, N / 2] = silu(gate) * up`` (``limit``, ``activation``:
+    the other activations of :func:`silu_mul`).
     ``row_stats`` (from :func:`linear_pair_residual`): ``x`` still lacks the division by its rows' root mean square,
     and the results are multiplied by it before they are rounded.
 
@@ -1560,7 +1619,7 @@ def linear_pair(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, add: b
                                   _i(1 if (PAIR_WIDE if wide is None else wide) else 0),
                                   _i(m), _i(n), _i(k), _ptr(row_stats.partials if row_stats else None),
                                   _i(row_stats.count if row_stats else 0), _f(row_stats.eps if row_stats else 0.0), None, None,
-                                  _i(0), None, _f(limit or 0.0), _ptr(device_error_flag(x.device)), _stream()))
+                                  _i(0), None, _i(_gate_code(activation, limit)), _f(limit or 0.0), _ptr(device_error_flag(x.device)), _stream()))
 
 
 QKV_IN_PRODUCT = __import__("os").environ.get("MINISERVE_B200_QKV_IN_PRODUCT", "1") == "1"
@@ -1881,7 +1940,8 @@ def wide_blocks(n: int, k: int) -> int:
 
 
 def _wide_call(x, weight, out, out_code: int, mode: int, m: int, n: int, k: int, row_stats: Optional[RowStats],
-               residual=None, norm_weight=None, x_next=None, out_partials=None, limit: Optional[float] = None) -> None:
+               residual=None, norm_weight=None, x_next=None, out_partials=None, limit: Optional[float] = None,
+               activation: str = "silu") -> None:
     if row_stats is not None:
         _want(row_stats.partials, "row_stats.partials", torch.float32)
         if row_stats.partials.dim() != 2 or row_stats.partials.shape[1] != 8 or row_stats.partials.shape[0] < row_stats.count:
@@ -1890,18 +1950,18 @@ def _wide_call(x, weight, out, out_code: int, mode: int, m: int, n: int, k: int,
         _ptr(x), _ptr(weight), _ptr(out), _i(out_code), _i(mode), _i(m), _i(n), _i(k),
         _ptr(row_stats.partials if row_stats else None), _i(row_stats.count if row_stats else 0),
         _f(row_stats.eps if row_stats else 0.0), _ptr(residual), _ptr(norm_weight),
-        _i(_code(norm_weight.dtype) if norm_weight is not None else 0), _ptr(x_next), _ptr(out_partials), _f(limit or 0.0),
+        _i(_code(norm_weight.dtype) if norm_weight is not None else 0), _ptr(x_next), _ptr(out_partials), _i(_gate_code(activation, limit)), _f(limit or 0.0),
         _ptr(device_error_flag(x.device)), _stream()))
 
 
 def linear_wide(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: bool = False,
-                row_stats: Optional[RowStats] = None, limit: Optional[float] = None) -> None:
+                row_stats: Optional[RowStats] = None, limit: Optional[float] = None, activation: str = "silu") -> None:
     """``out = x @ weight^T`` for up to 8 rows of bfloat16 ``x`` by the library's kernel for weights of many
     rows (no sum across blocks); ``out`` bfloat16 or float32.
 
     ``gated``: ``weight [2 I, K]`` holds a gated feed-forward's two projections in blocks of sixteen rows,
     eight gate rows followed by the up rows of the same features (:func:`interleave_gate_up`), and
-    ``out [M, I]`` bfloat16 receives ``silu(gate) * up`` (``limit``: the clamped activation of :func:`silu_mul`).  ``row_stats``: ``x`` comes from
+    ``out [M, I]`` bfloat16 receives ``silu(gate) * up`` (``limit``, ``activation``: the other activations of :func:`silu_mul`).  ``row_stats``: ``x`` comes from
     :func:`linear_wide_residual`; its rows' norm is completed on the results (before the activation).
     """
     m, k = x.shape
@@ -1909,7 +1969,7 @@ def linear_wide(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated:
     _want(x, "x", torch.bfloat16)
     _want(weight, "weight", torch.bfloat16, (n, k))
     _want(out, "out", torch.bfloat16 if gated else None, (m, n // 2 if gated else n))
-    _wide_call(x, weight, out, _code(out.dtype), 1 if gated else 0, m, n, k, row_stats, limit=limit)
+    _wide_call(x, weight, out, _code(out.dtype), 1 if gated else 0, m, n, k, row_stats, limit=limit, activation=activation)
 
 
 def linear_wide_residual(x: torch.Tensor, weight: torch.Tensor, residual: torch.Tensor, norm_weight: torch.Tensor,
@@ -2024,9 +2084,9 @@ WIDE_GATED_MIN_ROWS = 8192     # of the paired weight: the rule when nothing was
 
 
 def gated_up(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row_stats: Optional[RowStats] = None,
-             limit: Optional[float] = None) -> None:
-    """``out[M, I] = silu(x @ gate^T) * (x @ up^T)`` with ``weight = interleave_gate_up(gate, up)``; with ``limit`` the clamped
-    activation of :func:`silu_mul` on the two products.
+             limit: Optional[float] = None, activation: str = "silu") -> None:
+    """``out[M, I] = silu(x @ gate^T) * (x @ up^T)`` with ``weight = interleave_gate_up(gate, up)``; with ``limit`` or ``activation``
+    another activation of :func:`silu_mul` on the two products.
     (``row_stats``: see :func:`linear_wide`; the caller has asked :func:`fold_supported` first.)
 
     Few rows of bfloat16 go through :func:`linear_wide`, which applies the activation as it stores, where that
@@ -2038,21 +2098,22 @@ def gated_up(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row_stats
     _want(out, "out", x.dtype, (m, two_i // 2))
     if row_stats is not None:
         if row_stats.per_row:
-            linear_pair(x, weight, out, gated=True, row_stats=row_stats, limit=limit)
+            linear_pair(x, weight, out, gated=True, row_stats=row_stats, limit=limit, activation=activation)
         else:
-            linear_wide(x, weight, out, gated=True, row_stats=row_stats, limit=limit)
+            linear_wide(x, weight, out, gated=True, row_stats=row_stats, limit=limit, activation=activation)
         return
     if x.dtype == torch.bfloat16 and 0 < m <= SKINNY_MAX_ROWS and _gated_choice(x, weight) == "wide":
-        linear_wide(x, weight, out, gated=True, limit=limit)
+        linear_wide(x, weight, out, gated=True, limit=limit, activation=activation)
         return
     if x.dtype == torch.bfloat16 and k % 8 == 0 and pair_preferred(x.device, m, two_i, gated=True):
         choice = _pair_or_library("gated", m, weight)
         if choice != "library":
-            linear_pair(x, weight, out, gated=True, wide=choice == "wide", limit=limit)    # many rows: the activation is applied as the tiles are stored
+            # many rows: the activation is applied as the tiles are stored
+            linear_pair(x, weight, out, gated=True, wide=choice == "wide", limit=limit, activation=activation)
             return
     gate_up = torch.empty((m, two_i), dtype=x.dtype, device=x.device)
     linear(x, weight, gate_up)
-    silu_mul(gate_up, out, paired=True, limit=limit)
+    silu_mul(gate_up, out, paired=True, limit=limit, activation=activation)
 
 
 def _gated_choice(x: torch.Tensor, weight: torch.Tensor) -> str:

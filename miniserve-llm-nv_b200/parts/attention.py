@@ -12,8 +12,8 @@ All sizes are arguments.  ``window`` limits a query to the last ``window`` keys;
 overrides the score scale; ``position`` is a :class:`~.spec.PartSpec` of the position family.
 ``score_softcap`` c turns a scaled score s into ``c * tanh(s / c)`` and ``score_bias_slopes`` (one
 number per query head) adds ``slope * (key position - query position)`` to it: position
-encodings that act on the scores instead of on queries and keys.  Either of them selects the
-general attention kernel.
+encodings that act on the scores instead of on queries and keys.  Every attention kernel has the soft
+cap; the bias selects the general one.
 
 Further options, each off by default: ``value_dim`` (value heads of another size than query and key heads; the
 output projection then reads ``num_heads * value_dim`` numbers), ``sink`` (the softmax's denominator gets one more
@@ -36,7 +36,12 @@ are multiplied entry by entry by ``sigmoid(W_g x)``, a gate of ``num_heads * val
 ``query_temperature`` (coef, every) (the queries of position p are multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)``) with
 ``kernels.qkv_prepare_rows``, and ``conv_taps`` (q, k and v pass a short causal convolution per channel, ``<name><conv_suffix>`` of shape ``[channels, taps]``
 without bias, directly after the projection; the last ``taps - 1`` projected rows are the request's state, so
-``cache_need()`` is then the pair (pages, state)).
+``cache_need()`` is then the pair (pages, state)).  ``bias="qkv"``: biases on the q, k and v projections alone.
+
+``value_mix``: values shared along the depth of the model.  ``"keep"``: this layer leaves its tokens' values (biases included) for
+later layers of the step; ``"mix"``: the layer's values become ``(1 - share) v + share v_kept`` in float32 before they are
+cached, with ``share`` the layer's stored number ``mix_name`` (no dimensions) and ``v_kept`` what the layer with ``"keep"`` left for
+the same token.  Tokens of earlier steps need nothing: their mixed values are in the cache.
 """
 
 from __future__ import annotations
@@ -63,11 +68,11 @@ class Attention(Part):
                  output_gate: bool = False, own_kv: bool = True, gate_name: str = "g_proj.weight",
                  values_from_keys: bool = False, bias: bool = False, bias_suffix: str = ".b", qk_norm_weight: bool = True,
                  conv_taps: Optional[int] = None, conv_suffix: str = ".conv", sink_name: str = "sink",
-                 query_temperature: Optional[tuple] = None) -> None:
+                 query_temperature: Optional[tuple] = None, value_mix: Optional[str] = None, mix_name: str = "vmix") -> None:
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} key/value heads")
         general_form = bool(sink or output_gate or not own_kv or values_from_keys or (value_dim is not None and value_dim != head_dim)
-                            or bias or conv_taps or not qk_norm_weight or qk_norm == "row" or query_temperature is not None)
+                            or bias or conv_taps or not qk_norm_weight or qk_norm == "row" or query_temperature is not None or value_mix)
         if general_form and 1 <= head_dim <= kernels.MAX_HEAD_DIM:
             pass            # (the general form's kernels take odd head sizes too; the rotation checks its own size)
         elif head_dim % 2 or not 2 <= head_dim <= kernels.MAX_HEAD_DIM:
@@ -103,7 +108,14 @@ class Attention(Part):
             raise ValueError(f"output_gate is False, 'head' (True) or 'entry', not {output_gate!r}")
         self.sink, self.output_gate, self.own_kv = bool(sink), bool(output_gate), bool(own_kv)
         self.gate_per_entry = output_gate == "entry"
-        self.bias, self.qk_norm_weight = bool(bias), bool(qk_norm_weight)
+        if bias not in (False, True, "qkv"):
+            raise ValueError(f"bias is False, True (all four projections) or 'qkv', not {bias!r}")
+        self.bias, self.bias_on_output, self.qk_norm_weight = bool(bias), bias is True, bool(qk_norm_weight)
+        if value_mix not in (None, "keep", "mix"):
+            raise ValueError(f"value_mix is None, 'keep' or 'mix', not {value_mix!r}")
+        if value_mix and (not own_kv or values_from_keys or conv_taps or self.prepare_rows):
+            raise ValueError("values are shared between layers with values of their own, without convolutions and row norms")
+        self.value_mix, self.mix_share = value_mix, 0.0
         self.conv_taps = int(conv_taps) if conv_taps else None
         if self.conv_taps is not None and (not own_kv or values_from_keys or not 1 <= self.conv_taps <= kernels.MAX_CONV_TAPS):
             raise ValueError(f"conv_taps {conv_taps}: 1..{kernels.MAX_CONV_TAPS} taps on a layer's own queries, keys and values")
@@ -113,12 +125,13 @@ class Attention(Part):
         if self.values_from_keys and (self.value_dim != head_dim or not self.own_kv):
             raise ValueError("values_from_keys: the values are the layer's own keys, so both have the same size")
         self.general = (self.sink or self.output_gate or not self.own_kv or self.values_from_keys or self.value_dim != head_dim
-                        or self.bias or self.conv_taps is not None or not self.qk_norm_weight or self.prepare_rows)
-        if self.general and (self.score_softcap or self.score_bias_slopes is not None):
-            raise ValueError("score modifiers are not implemented together with value_dim, sink, output_gate or own_kv=False")
+                        or self.bias or self.conv_taps is not None or not self.qk_norm_weight or self.prepare_rows
+                        or self.value_mix is not None)
+        if self.general and self.score_bias_slopes is not None:
+            raise ValueError("a bias of the scores is not implemented together with value_dim, sink, output_gate or own_kv=False")
         self.names = dict(q=prefix + q_name, k=prefix + k_name, v=prefix + v_name, o=prefix + o_name,
                           q_norm=prefix + q_norm_name, k_norm=prefix + k_norm_name, g=prefix + gate_name,
-                          sink=prefix + sink_name)
+                          sink=prefix + sink_name, mix=prefix + mix_name)
         for key in ("q", "k", "v", "o"):
             self.names[key + "_b"] = self.names[key] + bias_suffix
             self.names[key + "_conv"] = self.names[key] + conv_suffix
@@ -158,7 +171,10 @@ class Attention(Part):
         specs.append(ParamSpec(self.names["o"], (h, self.num_heads * dv)))
         present = ["q"] + (["k"] if self.own_kv else []) + (["v"] if self.own_kv and not self.values_from_keys else [])
         if self.bias:
-            specs += [ParamSpec(self.names[key + "_b"], (self._rows_of(key),), "vector") for key in present + ["o"]]
+            specs += [ParamSpec(self.names[key + "_b"], (self._rows_of(key),), "vector")
+                      for key in present + (["o"] if self.bias_on_output else [])]
+        if self.value_mix == "mix":
+            specs.append(ParamSpec(self.names["mix"], (), "vector"))
         if self.conv_taps is not None:
             specs += [ParamSpec(self.names[key + "_conv"], (self._rows_of(key), self.conv_taps)) for key in present]
         return specs
@@ -204,7 +220,10 @@ class Attention(Part):
                 for key in present:
                     self.in_bias[at:at + self._rows_of(key)] = tensors[n[key + "_b"]].float()
                     at += self._rows_of(key)
-                self.o_bias = tensors[n["o_b"]].float().contiguous()
+                if self.bias_on_output:
+                    self.o_bias = tensors[n["o_b"]].float().contiguous()
+            if self.value_mix == "mix":
+                self.mix_share = float(tensors[n["mix"]])
             if self.conv_taps is not None:
                 self.conv_weight = torch.cat([tensors[n[key + "_conv"]].float() for key in present], dim=0).contiguous()
                 if self.in_bias is not None:
@@ -301,14 +320,16 @@ class Attention(Part):
                                      self.k_norm_weight, self.eps, cos_sin, rotary_dim, cache.key_pool, cache.value_pool, q,
                                      interleaved=interleaved, positions=ctx.positions, temperature=self.query_temperature)
         else:
+            kept = None if self.value_mix is None else ctx.buffer("attention.kept_values", (n, n_kv * dv), x.dtype)
             kernels.qkv_prepare(heads, 0, self.k_col, self.v_col, n_q, n_kv, d, dv, cache.slots, self.q_norm_weight,
                                 self.k_norm_weight, self.eps, cos_sin, rotary_dim, cache.key_pool, cache.value_pool, q,
-                                interleaved=interleaved, bias=self.in_bias if state is None else None)
+                                interleaved=interleaved, bias=self.in_bias if state is None else None, kept_values=kept,
+                                mix_share=self.mix_share if self.value_mix == "mix" else None)
         attended = ctx.buffer("attention.attended", (n, n_q, dv), x.dtype)
         per_head = self.output_gate and not self.gate_per_entry
         kernels.paged_attention(q, cache.key_pool, cache.value_pool, cache.block_tables, ctx.request_of_token,
                                 ctx.positions, ctx.query_start, ctx.context_lens, ctx.max_query_len,
-                                ctx.max_context_len, self.scale, self.window, attended, ctx.host_query_start or None,
+                                ctx.max_context_len, self.scale, self.window, attended, ctx.host_query_start or None, self.score_softcap,
                                 sink=self.sink_scores if self.learned_sink else self.sink, gate=proj if per_head else None, gate_col=max(self.gate_col, 0))
         if self.gate_per_entry:
             kernels.sigmoid_gate_mul(attended.view(n, n_q * dv), proj, self.gate_col, attended.view(n, n_q * dv))

@@ -1,5 +1,5 @@
 """Block arrangements.  ``pre_norm``: ``h += mixer(norm(h)); h += feed_forward(norm(h))``
-(miniserve/model/qwen3.py:336-346).  ``parallel``: one norm whose output both sublayers read,
+(miniserve/model/qwen3.py:336-346); a layer without a feed-forward is ``h += mixer(norm(h))``.  ``parallel``: one norm whose output both sublayers read,
 ``h += mixer(norm(h)) + feed_forward(norm(h))``; a layer without a feed-forward is ``h += mixer(norm(h))``.
 ``parallel_two_norms``: the same with a norm of its own for each sublayer, ``h += mixer(norm_1(h)) + feed_forward(norm_2(h))``.
 ``sandwich``: a norm on both sides of each sublayer, ``h += post(mixer(norm(h))); h += post(feed_forward(norm(h)))``.
@@ -61,11 +61,13 @@ class PreNormBlock:
     takes_next_block = True          # forward() has the `next_block` argument and may receive a FoldedInput as `pending`
 
     def __init__(self, *, mixer, feed_forward, mixer_norm, feed_forward_norm) -> None:
+        if (feed_forward is None) != (feed_forward_norm is None):
+            raise ValueError("a pre-norm block has a feed-forward with its norm, or neither")
         self.mixer, self.feed_forward = mixer, feed_forward
         self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
 
     def parts(self):
-        return [self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward]
+        return [part for part in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if part is not None]
 
     def forward(self, residual: torch.Tensor, pending: Pending, ctx: StepContext, cache: Any,
                 next_block: Any = None) -> Pending:
@@ -78,6 +80,8 @@ class PreNormBlock:
         else:
             normed = ctx.buffer("block.normed", tuple(residual.shape), ctx.dtype)
             self.mixer_norm.add_and_norm(residual, pending, normed)
+        if self.feed_forward is None:
+            return self._last_part(self.mixer, residual, ctx, next_block, normed, ctx, cache)
         fold = fold_between(self.mixer, self.feed_forward_norm, self.feed_forward, ctx)
         if fold is not None:
             normed = self.mixer.forward(normed, ctx, cache, fold=NormFold(residual, *fold))
@@ -88,13 +92,19 @@ class PreNormBlock:
                 delta = self.mixer.forward(normed, ctx, cache)
             normed = ctx.buffer("block.normed", tuple(residual.shape), ctx.dtype)      # (the mixer has read the first)
             self.feed_forward_norm.add_and_norm(residual, delta, normed)
+        return self._last_part(self.feed_forward, residual, ctx, next_block, normed, ctx)
+
+    @staticmethod
+    def _last_part(part, residual: torch.Tensor, ctx: StepContext, next_block: Any, *args) -> Pending:
+        """``part.forward(*args)`` for the layer's last sublayer: its last product prepares the next layer's input, or adds into
+        the stream, where both sides offer it."""
         if next_block is not None and getattr(next_block, "takes_next_block", False):
-            fold = fold_between(self.feed_forward, getattr(next_block, "mixer_norm", None), getattr(next_block, "mixer", None), ctx)
+            fold = fold_between(part, getattr(next_block, "mixer_norm", None), getattr(next_block, "mixer", None), ctx)
             if fold is not None:
-                return self.feed_forward.forward(normed, ctx, fold=NormFold(residual, *fold))
-        if adds_into_stream(self.feed_forward, ctx):
-            return self.feed_forward.forward(normed, ctx, fold=ResidualAdd(residual))
-        return self.feed_forward.forward(normed, ctx)
+                return part.forward(*args, fold=NormFold(residual, *fold))
+        if adds_into_stream(part, ctx):
+            return part.forward(*args, fold=ResidualAdd(residual))
+        return part.forward(*args)
 
 
 @register_block("parallel")

@@ -20,9 +20,12 @@ Other ways to route, each off by default:
   as it is (the weights of a token then do not add up to 1).  ``correction_name``: a vector added to the scores for the
   CHOICE only.
 * ``groups=(count, keep)``: the router's outputs form ``count`` equal groups of neighbours; a group's score is its
-  largest choice score, and only members of the ``keep`` best groups can be chosen.
+  largest choice score (``group_score="largest"``) or the sum of its two largest (``"two_largest"``), and only members of the
+  ``keep`` best groups can be chosen.
 * ``scoring="sigmoid"``: scores are ``sigmoid(z)`` of every router output on its own; the ``top`` largest are chosen (a tie
   goes to the lower index) and a chosen expert's weight is its score as it is.
+* ``normalize=e``: the chosen scores are divided by their sum plus ``e``; ``weight_scale``: the weights are multiplied by a
+  constant (after that).  Both for scores of either kind over all outputs.
 * ``weight_on="input"``: the weight multiplies what the expert reads, not what it returns: the output is the sum of
   ``expert(w h)`` over the chosen experts.  (An expert's first products are linear, so the factor is applied to their
   float32 sums as the activation is formed.)
@@ -56,7 +59,8 @@ class RoutedExperts(Part):
                  shared_name: str = "shared.", up_name: str = "up", down_name: str = "down", gate_name: str = "gate",
                  limit: Optional[float] = None, shared_limit: Optional[float] = None, identity: int = 0,
                  scoring: str = "chosen_softmax", correction_name: Optional[str] = None, groups: tuple = (1, 1),
-                 shared_gate_name: Optional[str] = None, weight_on: str = "output") -> None:
+                 shared_gate_name: Optional[str] = None, weight_on: str = "output", group_score: str = "largest",
+                 normalize: Optional[float] = None, weight_scale: float = 1.0) -> None:
         if activation not in ("relu_square", "clamped_glu", "silu_glu"):
             raise ValueError(f"routed_experts implements the activations 'relu_square', 'clamped_glu' and 'silu_glu', not {activation!r}")
         if scoring not in ("chosen_softmax", "all_softmax", "sigmoid"):
@@ -76,7 +80,13 @@ class RoutedExperts(Part):
         if activation == "silu_glu" and shared_size:
             raise ValueError("a shared expert is not implemented for the 'silu_glu' activation")
         if (correction_name or (count, keep) != (1, 1)) and scoring not in ("all_softmax", "sigmoid"):
-            raise ValueError("a correction of the choice and groups are implemented for scoring='all_softmax'")
+            raise ValueError("a correction of the choice and groups are implemented for scoring='all_softmax' and 'sigmoid'")
+        if group_score not in kernels.GROUP_SCORES:
+            raise ValueError(f"a group is scored by {' or '.join(kernels.GROUP_SCORES)}, not {group_score!r}")
+        if (normalize is not None or weight_scale != 1.0) and scoring == "chosen_softmax":
+            raise ValueError("normalized or scaled weights are implemented for scoring='all_softmax' and 'sigmoid'")
+        self.group_score, self.weight_scale = group_score, float(weight_scale)
+        self.normalize = None if normalize is None else float(normalize)
         self.prefix, self.hidden_size = prefix, hidden_size
         self.experts, self.top, self.expert_size, self.shared_size = experts, top, expert_size, shared_size
         self.identity, self.total, self.scoring, self.groups = identity, total, scoring, (count, keep)
@@ -153,7 +163,8 @@ class RoutedExperts(Part):
         weights = ctx.buffer("experts.weights", (n, top), torch.float32)
         logits = ctx.buffer("experts.logits", (n, self.router_weight.shape[0]), torch.float32)
         kernels.router_topk(x, self.router_weight, self.router_b, top, ids, weights, logits, choose_from=self.total,
-                            scoring=self.scoring, correction=self.correction, groups=self.groups)
+                            scoring=self.scoring, correction=self.correction, groups=self.groups, group_score=self.group_score,
+                            normalize=self.normalize, weight_scale=self.weight_scale)
         offsets = ctx.buffer("experts.offsets", (self.total + 1,), torch.int32)
         order = ctx.buffer("experts.order", (pairs,), torch.int32)
         place = ctx.buffer("experts.place", (pairs,), torch.int32)

@@ -1,5 +1,5 @@
 """Feed-forward parts.  ``gated_mlp``: ``down(act(gate(x)) * up(x))`` without biases
-(miniserve/model/layers.py:71-87) with ``silu`` as the activation, or, ``clamped_glu`` with ``limit``, ``down(g sigmoid(1.702 g) (u +
+(miniserve/model/layers.py:71-87) with ``silu`` or ``gelu_tanh`` (the tanh form of GELU, no biases) as the activation, or, ``clamped_glu`` with ``limit``, ``down(g sigmoid(1.702 g) (u +
 1))`` with ``g = min(gate(x), limit)`` and ``u = clamp(up(x), -limit, limit)``; gate and up run as one
 matrix product over one weight that holds both.  Where the intermediate size is a multiple of eight
 the rows of the two alternate in blocks of eight (``kernels.interleave_gate_up``), which lets the
@@ -25,10 +25,13 @@ class GatedMLP(Part):
                  gate_name: str = "gate_proj.weight", up_name: str = "up_proj.weight",
                  down_name: str = "down_proj.weight", bias: bool = False, limit: Optional[float] = None,
                  gate_bias_name: str = "gate_proj.bias", up_bias_name: str = "up_proj.bias", down_bias_name: str = "down_proj.bias") -> None:
-        if activation not in ("silu", "clamped_glu"):
-            raise ValueError(f"gated_mlp implements the activations 'silu' and 'clamped_glu', not {activation!r}")
+        if activation not in ("silu", "clamped_glu", "gelu_tanh"):
+            raise ValueError(f"gated_mlp implements the activations 'silu', 'gelu_tanh' and 'clamped_glu', not {activation!r}")
+        if activation == "gelu_tanh" and bias:
+            raise ValueError("gated_mlp: biases are implemented for the 'silu' activation")
+        self.activation = activation
         if (activation == "clamped_glu") != (limit is not None) or (limit is not None and (limit <= 0 or bias)):
-            raise ValueError(f"gated_mlp: 'clamped_glu' takes a limit above 0 and no biases, 'silu' no limit (limit {limit}, bias {bias})")
+            raise ValueError(f"gated_mlp: 'clamped_glu' takes a limit above 0 and no biases, the others no limit (limit {limit}, bias {bias})")
         self.limit = None if limit is None else float(limit)
         self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
         self.names = dict(gate=prefix + gate_name, up=prefix + up_name, down=prefix + down_name,
@@ -82,7 +85,7 @@ class GatedMLP(Part):
         out = ctx.buffer("gated_mlp.out", (n, self.hidden_size), x.dtype)
         if self.paired:
             hidden = ctx.buffer("gated_mlp.hidden", (n, self.intermediate_size), x.dtype)
-            kernels.gated_up(x, self.gate_up_weight, hidden, row_stats=stats, limit=self.limit)
+            kernels.gated_up(x, self.gate_up_weight, hidden, row_stats=stats, limit=self.limit, activation=self.activation)
             if isinstance(fold, ResidualAdd):
                 kernels.linear_add(hidden, self.down_weight, fold.residual)
                 return None
@@ -100,9 +103,9 @@ class GatedMLP(Part):
                 kernels.silu_mul(gate_up, hidden, bias=self.gate_up_bias)
                 kernels.linear(hidden, self.down_weight, out)
                 kernels.add_bias(out, self.down_bias)
-            elif self.limit is not None:
+            elif self.activation != "silu":
                 hidden = ctx.buffer("gated_mlp.hidden", (n, self.intermediate_size), x.dtype)
-                kernels.silu_mul(gate_up, hidden, limit=self.limit)
+                kernels.silu_mul(gate_up, hidden, limit=self.limit, activation=self.activation)
                 kernels.linear(hidden, self.down_weight, out)
             else:
                 kernels.gated_linear(gate_up, self.down_weight, out)

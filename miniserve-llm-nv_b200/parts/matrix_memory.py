@@ -30,6 +30,11 @@ the decay's and the output gate's projections products of two matrices through r
 v_t^T`` with a constant of the head, ``o_t = S_t^T q_t``; the concatenated heads are divided by their root mean square TOGETHER,
 multiplied by a weight and by ``sigmoid(W_g h)``; ``W_o`` maps the result back.
 
+``gated_linear_attention``: ``q = W_q h * d^(-1/2)``, ``k = W_k h``, ``v = W_v h``, per head and KEY channel a decay ``a_t = sigmoid(W_a2
+W_a1 h + b)^(1 / tau)`` through ``rank`` numbers; ``S_t = diag(a_t) S_(t-1) + k_t v_t^T``, ``o_t = S_t^T q_t``; every head's ``o`` is
+divided by its root mean square, multiplied by a weight over ``dv`` that the heads share and by ``silu(W_g h)``; ``W_o`` maps the
+result back.
+
 What a request carries from token to token is one float32 vector per layer (:class:`~.base.StateNeed`, zero at
 admission): for ``matrix_memory`` the heads' matrices with ``n`` as one more column, then the heads' maxima; for
 ``delta_rule`` the convolution's last ``taps - 1`` inputs, then the heads' matrices.  Gates, decays, step sizes, unit
@@ -276,5 +281,61 @@ class LinearAttention(Part):
         # (the heads are normed together: one "head" of H * dv entries)
         kernels.head_norm_gate(y.view(n, 1, H * dv), None, self.norm_weight, proj, self.g_col, "sigmoid", self.eps, gated)
         out = ctx.buffer("linear_attention.out", (n, self.hidden_size), x.dtype)
+        kernels.linear(gated, self.o_weight, out)
+        return out
+
+
+@register_mixer("gated_linear_attention")
+class GatedLinearAttention(Part):
+    def __init__(self, *, prefix: str, hidden_size: int, heads: int, head_dim: int, value_dim: int, rank: int, tau: float, eps: float,
+                 q_name: str = "q", k_name: str = "k", v_name: str = "v", g_name: str = "g", o_name: str = "o", norm_name: str = "norm",
+                 a_name: str = "a", bias_suffix: str = ".b") -> None:
+        if min(hidden_size, heads, head_dim, value_dim, rank) < 1 or not tau > 0:
+            raise ValueError("gated_linear_attention: every size and tau must be positive")
+        if head_dim > kernels.MAX_MATRIX_SCAN_DIM or rank > kernels.MAX_EXPAND_RANK:
+            raise ValueError(f"gated_linear_attention: keys of {head_dim} entries (at most {kernels.MAX_MATRIX_SCAN_DIM}), a decay through "
+                             f"{rank} numbers (at most {kernels.MAX_EXPAND_RANK})")
+        self.hidden_size, self.heads, self.head_dim, self.value_dim, self.rank = hidden_size, heads, head_dim, value_dim, rank
+        self.tau, self.eps = float(tau), float(eps)
+        self.q_col, self.k_col, self.v_col = 0, heads * head_dim, 2 * heads * head_dim
+        self.g_col = self.v_col + heads * value_dim
+        self.names = {key: prefix + name for key, name in dict(
+            q=q_name, k=k_name, v=v_name, g=g_name, o=o_name, norm=norm_name, a1=a_name + "1", a2=a_name + "2",
+            a_b=a_name + "2" + bias_suffix).items()}
+        self.in_weight = self.decay_weight = self.decay_expand = self.decay_bias = self.norm_weight = self.o_weight = None
+
+    def param_specs(self) -> list[ParamSpec]:
+        n, h, H, d, dv = self.names, self.hidden_size, self.heads, self.head_dim, self.value_dim
+        return [ParamSpec(n["q"], (H * d, h)), ParamSpec(n["k"], (H * d, h)), ParamSpec(n["v"], (H * dv, h)),
+                ParamSpec(n["g"], (H * dv, h)), ParamSpec(n["o"], (h, H * dv)), ParamSpec(n["norm"], (dv,), "vector"),
+                ParamSpec(n["a1"], (self.rank, h), "matrix_f32"), ParamSpec(n["a2"], (H * d, self.rank), "matrix_f32"),
+                ParamSpec(n["a_b"], (H * d,), "vector")]
+
+    def cache_need(self) -> StateNeed:
+        return StateNeed((self.heads * self.value_dim * self.head_dim,), torch.float32)
+
+    def load(self, tensors: dict[str, torch.Tensor]) -> None:
+        n = self.names
+        self.in_weight = _pad_rows([tensors[n["q"]], tensors[n["k"]], tensors[n["v"]], tensors[n["g"]]], self.hidden_size)
+        self.decay_weight = tensors[n["a1"]].float().contiguous()
+        self.decay_expand = tensors[n["a2"]].float().t().contiguous()          # [rank, H * d]: the kernel reads it transposed
+        self.decay_bias = tensors[n["a_b"]].float().contiguous()
+        self.norm_weight = tensors[n["norm"]].float().contiguous()
+        self.o_weight = tensors[n["o"]]
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: StateView) -> torch.Tensor:
+        n, H, d, dv = x.shape[0], self.heads, self.head_dim, self.value_dim
+        proj = ctx.buffer("gated_linear_attention.proj", (n, self.in_weight.shape[0]), x.dtype)
+        kernels.linear(x, self.in_weight, proj)
+        mid = ctx.buffer("gated_linear_attention.mid", (n, self.rank), torch.float32)
+        kernels.small_linear_f32(x, self.decay_weight, None, mid)
+        decays = ctx.buffer("gated_linear_attention.decays", (n, H * d), torch.float32)
+        kernels.low_rank_expand(mid, 0, self.decay_expand, decays, bias=self.decay_bias, tau=self.tau)
+        y = ctx.buffer("gated_linear_attention.y", (n, H, dv), torch.float32)
+        kernels.matrix_scan("channel_decay", proj, self.q_col, proj, self.k_col, proj, self.v_col, None, cache.states, 0,
+                            ctx.state_slots, ctx.query_start, ctx.max_query_len, H, H, d, dv, y, q_scale=d ** -0.5, channel_decay=decays)
+        gated = ctx.buffer("gated_linear_attention.gated", (n, H * dv), x.dtype)
+        kernels.head_norm_gate(y, None, self.norm_weight, proj, self.g_col, "silu", self.eps, gated)
+        out = ctx.buffer("gated_linear_attention.out", (n, self.hidden_size), x.dtype)
         kernels.linear(gated, self.o_weight, out)
         return out

@@ -3,7 +3,8 @@
 lies around zero and stands for ``1 + weight`` (added once, in float32, when the weight is loaded).  ``identity``: no norm
 at all, for blocks whose sublayers read the residual stream itself: what is pending is added and the stream is handed on in
 the compute type.  ``layer``: layer norm with weight and bias, ``weight * (x - mean) / sqrt(mean((x - mean)^2) + eps) + bias``;
-two of them that read the same stream run as one kernel (``add_and_norm_both``)."""
+two of them that read the same stream run as one kernel (``add_and_norm_both``).  ``dynamic_tanh``: no statistics at all, entry by
+entry ``weight * tanh(alpha * x) + bias`` with one ``alpha`` per norm."""
 
 from __future__ import annotations
 
@@ -133,3 +134,37 @@ class LayerNorm(Part):
         first, second, vector = self._pending(delta)
         kernels.add_layernorm(residual, first, self.weight, self.bias, self.eps, out, None, second, vector, other.weight, other.bias,
                               other_out)
+
+
+@register_norm("dynamic_tanh")
+class DynamicTanh(Part):
+    """``weight * tanh(alpha * x) + bias`` (``name``, ``name + alpha_suffix`` without dimensions, ``name + bias_suffix``), in float32."""
+
+    def __init__(self, *, name: str, size: int, prefix: str = "", alpha_suffix: str = ".alpha", bias_suffix: str = ".b") -> None:
+        self.name, self.size = prefix + name, size
+        self.alpha_name, self.bias_name = self.name + alpha_suffix, self.name + bias_suffix
+        self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+        self.alpha = 0.0
+
+    def param_specs(self) -> list[ParamSpec]:
+        return [ParamSpec(self.name, (self.size,), "vector"), ParamSpec(self.bias_name, (self.size,), "vector"),
+                ParamSpec(self.alpha_name, (), "vector")]
+
+    def load(self, tensors: dict[str, torch.Tensor]) -> None:
+        self.weight, self.bias = tensors[self.name].float().contiguous(), tensors[self.bias_name].float().contiguous()
+        self.alpha = float(tensors[self.alpha_name])
+
+    def add_and_norm(self, residual: torch.Tensor, delta, out: torch.Tensor,
+                     rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``residual += delta`` (float32, in place), ``out = norm(residual)``, as :meth:`RMSNorm.add_and_norm`."""
+        second = None
+        if isinstance(delta, StreamVector):
+            kernels.add_bias(residual, delta.vector)
+            delta = None
+        if isinstance(delta, tuple):
+            delta, second = delta
+        if delta is not None and not isinstance(delta, torch.Tensor):
+            raise TypeError(f"the dynamic tanh norm adds outputs or a vector, not {type(delta).__name__}")
+        kernels.add_dynamic_tanh(residual, delta, self.alpha, self.weight, self.bias, out, rows, second)
+        return out

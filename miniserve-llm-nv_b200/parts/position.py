@@ -4,8 +4,8 @@
 half-split pairing ``(j, j + rotary_dim/2)`` by default, interleaved pairing ``(2j, 2j+1)`` or
 a rotary size below the head size as options.  Angles, cosines and sines are float32 and are
 computed once per step for all layers that share the same encoding.  With ``scaling`` the
-frequencies are stretched the YaRN way (see :func:`scaled_frequencies`) and cosines and sines get a
-common magnitude.
+frequencies are stretched the YaRN way (see :func:`scaled_frequencies`), with cosines and sines getting a
+common magnitude, or by wavelength (see :func:`wavelength_frequencies`); which of the two, the constants' names say.
 ``none``: no position encoding.
 
 A position part either offers ``fused_args(ctx)``, the arguments of the fused
@@ -48,6 +48,26 @@ def scaled_frequencies(dims: int, theta: float, factor: float, original: float, 
     return frequencies, 0.1 * math.log(factor) + 1.0
 
 
+def wavelength_frequencies(dims: int, theta: float, factor: float, low: float, high: float, original: float) -> list:
+    """The frequencies ``f_i = theta^(-2i/dims)`` scaled by wavelength ``l_i = 2 pi / f_i`` (the Llama 3.1 way): short waves, ``l <
+    original / high``, stay; long ones, ``l > original / low``, are slowed down by ``factor``; between the two the share ``s =
+    (original / l - low) / (high - low)`` stays: ``(1 - s) f / factor + s f``.  In double precision, rounded by the caller."""
+    frequencies = []
+    for i in range(dims // 2):
+        f = theta ** (-2.0 * i / dims)
+        wavelength = 2.0 * math.pi / f
+        if wavelength > original / low:
+            f = f / factor
+        elif wavelength >= original / high:
+            stays = (original / wavelength - low) / (high - low)
+            f = (1.0 - stays) * f / factor + stays * f
+        frequencies.append(f)
+    return frequencies
+
+
+SCALINGS = {"yarn": ("factor", "original", "fast", "slow"), "wavelength": ("factor", "low", "high", "original")}
+
+
 @register_position("rope")
 class RotaryPosition(Part):
     def __init__(self, *, head_dim: int, theta: float, rotary_dim: Optional[int] = None,
@@ -59,8 +79,14 @@ class RotaryPosition(Part):
         self.interleaved = bool(interleaved)
         if self.rotary_dim % 2 or not 0 < self.rotary_dim <= head_dim:
             raise ValueError(f"rotary size {self.rotary_dim} must be even and within the head size {head_dim}")
-        # ``scaling``: the mapping {factor, original, fast, slow} of :func:`scaled_frequencies`, or None
-        self.scaling = None if not scaling else tuple(float(scaling[key]) for key in ("factor", "original", "fast", "slow"))
+        # ``scaling``: the mapping {factor, original, fast, slow} of :func:`scaled_frequencies` or {factor, low, high, original} of
+        # :func:`wavelength_frequencies`, or None; kept as (kind, constants)
+        self.scaling = None
+        if scaling:
+            kind = next((kind for kind, keys in SCALINGS.items() if set(keys) == set(scaling)), None)
+            if kind is None:
+                raise ValueError(f"a scaling has the constants {' or '.join(map(str, SCALINGS.values()))}, not {sorted(scaling)}")
+            self.scaling = (kind, tuple(float(scaling[key]) for key in SCALINGS[kind]))
         # "float32": the frequencies come from float32 arithmetic (rope.py:24-25); "float64": theta^(-2i/dims) is
         # computed in double precision and rounded to float32 once
         if frequencies not in ("float32", "float64"):
@@ -73,7 +99,11 @@ class RotaryPosition(Part):
         """``1 / theta ** (arange(0, rotary_dim, 2) / rotary_dim)`` in float32 (rope.py:24-25), or the scaled frequencies."""
         if self._inv_freq is None or self._inv_freq.device != torch.device(device):
             if self.scaling is not None:
-                frequencies, self.magnitude = scaled_frequencies(self.rotary_dim, self.theta, *self.scaling)
+                kind, constants = self.scaling
+                if kind == "yarn":
+                    frequencies, self.magnitude = scaled_frequencies(self.rotary_dim, self.theta, *constants)
+                else:
+                    frequencies = wavelength_frequencies(self.rotary_dim, self.theta, *constants)
                 self._inv_freq = torch.tensor(frequencies, dtype=torch.float64).to(torch.float32).to(device)
             elif self.frequencies == "float64":
                 exact = [self.theta ** (-2.0 * i / self.rotary_dim) for i in range(self.rotary_dim // 2)]

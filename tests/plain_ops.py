@@ -96,7 +96,7 @@ def qk_norm_rope_append(qkv, slots, q_weight, k_weight, eps, cos_sin, rotary_dim
         v_pool[page, :, offset, :] = v[token].to(v_pool.dtype)
 
 
-def silu_mul(gate_up, out, paired=False, bias=None, limit=None):
+def silu_mul(gate_up, out, paired=False, bias=None, limit=None, activation="silu"):
     n, inter = out.shape
     if bias is not None:
         gate_up = gate_up.double() + bias.double()
@@ -105,6 +105,9 @@ def silu_mul(gate_up, out, paired=False, bias=None, limit=None):
         g, u = blocks[:, :, 0].reshape(n, inter).double(), blocks[:, :, 1].reshape(n, inter).double()
     else:
         g, u = gate_up[:, :inter].double(), gate_up[:, inter:].double()
+    if activation == "gelu_tanh":
+        out.copy_((gelu_tanh(g) * u).to(out.dtype))
+        return
     out.copy_((clamped_glu_values(g, u, limit) if limit else g * torch.sigmoid(g) * u).to(out.dtype))
 
 
@@ -114,11 +117,11 @@ def _row_factor(row_stats, size):
     return 1.0 / torch.sqrt(total / size + row_stats.eps)
 
 
-def gated_up(x, weight, out, row_stats=None, limit=None):
+def gated_up(x, weight, out, row_stats=None, limit=None, activation="silu"):
     gate_up = x.double() @ weight.double().T
     if row_stats is not None:
         gate_up = gate_up * _row_factor(row_stats, x.shape[1])[:x.shape[0], None]
-    silu_mul(gate_up.to(x.dtype), out, paired=True, limit=limit)
+    silu_mul(gate_up.to(x.dtype), out, paired=True, limit=limit, activation=activation)
 
 
 FOLD_BLOCKS = 3     # the plain stand-in leaves its sums of squares in this many rows, as a kernel of three blocks would
@@ -266,7 +269,7 @@ def linear_batched(x, weight, out):
 
 
 def router_topk(x, weight, bias, top, ids, weights, scratch=None, *, choose_from=None, scoring="chosen_softmax",
-                correction=None, groups=(1, 1)):
+                correction=None, groups=(1, 1), group_score="largest", normalize=None, weight_scale=1.0):
     logits = x.double() @ weight.double().T
     if bias is not None:
         logits = logits + bias.double()
@@ -279,13 +282,17 @@ def router_topk(x, weight, bias, top, ids, weights, scratch=None, *, choose_from
         choice = scores if correction is None else scores + correction.double()
         count, keep = groups
         if keep < count:
-            best = choice.view(n, count, total // count).max(dim=2).values
+            ranked = choice.view(n, count, total // count).sort(dim=2, descending=True).values
+            best = ranked[:, :, :2].sum(dim=2) if group_score == "two_largest" else ranked[:, :, 0]
             kept = torch.zeros(n, count, dtype=torch.bool)
             kept.scatter_(1, best.sort(dim=1, descending=True, stable=True).indices[:, :keep], True)
             choice = choice.masked_fill(~kept[:, :, None].expand(n, count, total // count).reshape(n, total), -math.inf)
         chosen = choice.sort(dim=1, descending=True, stable=True).indices[:, :top]
         ids.copy_(chosen.to(ids.dtype))
-        weights.copy_(torch.gather(scores, 1, chosen).to(weights.dtype))
+        taken = torch.gather(scores, 1, chosen)
+        if normalize is not None:
+            taken = taken / (taken.sum(dim=1, keepdim=True) + normalize)
+        weights.copy_((taken * weight_scale).to(weights.dtype))
         return
     ranked = logits.sort(dim=1, descending=True, stable=True)
     ids.copy_(ranked.indices[:, :top].to(ids.dtype))
@@ -374,7 +381,7 @@ def postnorm_add_rmsnorm(residual, delta, post_weight, post_eps, weight, eps, ou
 
 
 def qkv_prepare(proj, q_col, k_col, v_col, n_q, n_kv, head_dim, value_dim, slots, q_weight, k_weight, eps, cos_sin,
-                rotary_dim, k_pool, v_pool, q_out, interleaved=False, bias=None, value_heads=None):
+                rotary_dim, k_pool, v_pool, q_out, interleaved=False, bias=None, value_heads=None, kept_values=None, mix_share=None):
     n = proj.shape[0]
     if bias is not None:
         proj = proj.double() + bias.double()
@@ -392,7 +399,12 @@ def qkv_prepare(proj, q_col, k_col, v_col, n_q, n_kv, head_dim, value_dim, slots
         return
     k = heads(k_col, n_kv, head_dim, k_weight)
     value_heads = n_kv if value_heads is None else value_heads
-    v = proj[:, v_col:v_col + value_heads * value_dim].view(n, value_heads, value_dim)
+    v = proj[:, v_col:v_col + value_heads * value_dim]
+    if mix_share is not None:
+        v = (1.0 - mix_share) * v.double() + mix_share * kept_values.double()
+    elif kept_values is not None:
+        kept_values.copy_(v.to(kept_values.dtype))
+    v = v.view(n, value_heads, value_dim)
     page_size = k_pool.shape[2]
     for token in range(n):
         slot = int(slots[token])
@@ -442,6 +454,18 @@ def add_layernorm(residual, delta, weight, bias, eps, out, rows=None, delta2=Non
     out.copy_((weight.double() * y + bias.double()).to(out.dtype))
     if out2 is not None:
         out2.copy_((weight2.double() * y + bias2.double()).to(out2.dtype))
+
+
+def add_dynamic_tanh(residual, delta, alpha, weight, bias, out, rows=None, delta2=None):
+    x = residual.double()
+    if delta is not None:
+        x = x + (delta.double() if delta2 is None else delta.double() + delta2.double())
+        if rows is None:
+            residual.copy_(x.to(residual.dtype))
+            x = residual.double()
+    if rows is not None:
+        x = x[rows.long()]
+    out.copy_((torch.tanh(alpha * x) * weight.double() + bias.double()).to(out.dtype))
 
 
 def stream_to_columns(residual, delta, out, col, delta2=None):
@@ -574,6 +598,10 @@ def matrix_scan(mode, q, q_col, k, k_col, v, v_col, gates, states, state_offset,
                 S = gates.double()[:, None, None] * S + vt[:, :, None] * kt[:, None, :]
                 y[t] = torch.einsum("hcd,hd->hc", S, qt).to(y.dtype)
                 continue
+            if mode == "channel_decay":
+                S = channel_decay[t].double().view(heads, 1, dim) * S + vt[:, :, None] * kt[:, None, :]
+                y[t] = torch.einsum("hcd,hd->hc", S, qt).to(y.dtype)
+                continue
             if mode == "channel_delta":
                 beta = torch.sigmoid(gates[t, gate_col:gate_col + heads].double())
                 S = channel_decay[t].double().view(heads, 1, dim) * S
@@ -641,11 +669,13 @@ def softplus(x):
     return torch.clamp(x, min=0.0) + torch.log1p(torch.exp(-x.abs()))
 
 
-def low_rank_expand(mid, col, weight_t, out, a_log=None, bias=None, per_head=0):
+def low_rank_expand(mid, col, weight_t, out, a_log=None, bias=None, per_head=0, tau=None):
     rank = weight_t.shape[0]
     value = mid[:, col:col + rank].double() @ weight_t.double()
     if a_log is not None:
         value = torch.exp(-torch.exp(a_log.double()).repeat_interleave(per_head) * softplus(value + bias.double()))
+    elif tau is not None:
+        value = torch.sigmoid(value + bias.double()).pow(1.0 / tau)
     out.copy_(value.to(out.dtype))
 
 
@@ -716,7 +746,7 @@ def install(monkeypatch) -> None:
                  "selective_scan", "gated_group_norm", "causal_conv", "add_bias", "scaled_sum", "small_linear_f32",
                  "unit_norm_heads", "exponential_gates", "decay_gates", "matrix_scan", "head_norm_gate", "gated_recurrence_scan",
                  "low_rank_expand", "channel_decays", "normed_sum", "sigmoid_gate_mul", "differential_combine", "token_shift",
-                 "pair_embedding", "qkv_prepare_rows", "add_layernorm", "stream_to_columns"):
+                 "pair_embedding", "qkv_prepare_rows", "add_layernorm", "add_dynamic_tanh", "stream_to_columns"):
         monkeypatch.setattr(kernels, name, globals()[name])
     monkeypatch.setattr(kernels, "attention_kernels", lambda *sizes: {"decode": "plain", "prompt": "plain"})
     monkeypatch.setattr(kernels, "latent_attention_kernels", lambda *sizes: {"decode": "plain", "prompt": "plain"})
