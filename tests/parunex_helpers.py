@@ -1,6 +1,6 @@
 """Small Parunex configurations for the tests, with weights made so that every tensor of the design moves its formula: alphas, weights
 and biases of the norms away from their neutral values, sinks between -1.5 and 2.5, biases of the size of the projections, shares of
-the kept values from slightly negative to one, decays that remember a dozen tokens or more and differ from channel to channel, and
+the kept values some of them negative, decays that remember a dozen tokens or more and differ from channel to channel, and
 routers whose choices are clear whatever the rounding."""
 
 from __future__ import annotations
@@ -49,9 +49,9 @@ def model(vocab, width, scale, eps, layers):
 # Sizes that differ from one another everywhere; three attention layers of which the last two take the first one's values (as four
 # heads of 12 in one of them and as two of 24 in the others); frequencies of all three kinds; a layer without a feed-forward.
 PARUNEX_A = model(203, 96, 3.0, 1e-5, [
-    layer(attention(4, 2, 16, 24, 0.3, rot(500.0, 12, (4.0, 1.0, 4.0, 64)), 5.0), moe(6, 2, 20, 1.7, 3, 2)),
+    layer(attention(4, 2, 16, 24, 0.3, rot(500.0, 12, (4.0, 1.0, 4.0, 64)), 1.5), moe(6, 2, 20, 1.7, 3, 2)),
     layer(gla(3, 20, 12, 16.0, 5), dense(56)),
-    layer(attention(8, 4, 20, 12, 0.25, rot(10000.0, 20), 3.0), None),
+    layer(attention(8, 4, 20, 12, 0.25, rot(10000.0, 20), 2.0), None),
     layer(gla(2, 12, 28, 4.0, 9), moe(8, 3, 24, 0.6, 2, 1)),
     layer(attention(6, 2, 24, 24, 0.2, rot(300.0, 8, (2.0, 2.0, 5.0, 40)), None), dense(44)),
 ])
@@ -145,7 +145,7 @@ def shape_weights(tensors: dict, config: dict) -> None:
                 put(p + f"mix.{name}.b", _normal(tuple(tensors[p + f"mix.{name}.b"].shape), seed + 10 + k, 0.4))
             put(p + "mix.g", _normal(tuple(tensors[p + "mix.g"].shape), seed + 14, width ** -0.5))
             if p + "mix.vmix" in tensors:
-                put(p + "mix.vmix", torch.tensor([0.6, -0.1, 1.0][index % 3]))
+                put(p + "mix.vmix", torch.tensor([0.6, -0.2, 0.8][index % 3]))
         else:
             put(p + "mix.norm", _normal((m["vdim"],), seed + 20, 0.3, 1.0))
             put(p + "mix.a1", _normal(tuple(tensors[p + "mix.a1"].shape), seed + 21, width ** -0.5))
