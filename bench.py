@@ -556,6 +556,21 @@ def _venarax(width, latent, window, sink, ff, vocab):
                 layers=[dict(mixer, mlp=mlp) for mixer in (windowed, full, windowed, full)])
 
 
+def _parunex(width, attention, recurrence, dense_ff, experts, top, count, keep, expert_ff, vocab):
+    """Four layers: gated linear attention with a gated feed-forward, capped attention with experts, the same two again; the second
+    attention layer mixes in the first one's values."""
+    heads, kv_heads, dim, vdim = attention
+    capped = dict(type="attention", mixer=dict(
+        heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=dim ** -0.5, softcap=50.0, v_mix=True,
+        rot=dict(base=500000.0, dims=dim, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))))
+    r_heads, r_dim, r_vdim, rank = recurrence
+    linear = dict(type="gla", mixer=dict(heads=r_heads, dim=r_dim, vdim=r_vdim, tau=16.0, rank=rank))
+    dense = dict(kind="dense", ff=dense_ff)
+    moe = dict(kind="moe", expert=dict(ff=expert_ff), router=dict(experts=experts, top=top, scale=2.5, groups=dict(count=count, keep=keep)))
+    return dict(architecture="Parunex", vocab=vocab, width=width, embedding=dict(scale=float(width) ** 0.5), norm=dict(eps=1e-6),
+                layers=[dict(linear, mlp=dense), dict(capped, mlp=moe), dict(linear, mlp=dense), dict(capped, mlp=moe)])
+
+
 # Layer sizes that resemble real models' (random weights, four layers each: two with a gated MLP, two with experts), and
 # the Qwen3 layers of equal width, head count and inner size beside them.
 DESIGN_SIZES = {
@@ -606,11 +621,24 @@ DESIGN_SIZES = {
     "windowed-lite": dict(venarax=_venarax(2048, (16, 128, 64, 128, 512), 512, (32, 8, 64, 64), 10944, 32000),
                           vesidra=_vesidra(2048, 6, _latent(16, 128, 64, 128, 512), 10944, 0, 0, 0, 0, 32000), depth=6,
                           qwen3=dict(hidden_size=2048, intermediate_size=10944, num_attention_heads=32, num_key_value_heads=8, head_dim=64)),
+    # Parunex: a gated linear attention of sixteen heads (keys and values of 128, decays through 16 numbers) with a feed-forward of
+    # 6,144, and sixteen heads of 128 over four key heads with capped scores and 16 experts of 1,024 (four per token, two of four
+    # groups); beside it Bafavik (the closest recurrences: constant decays and decays per key channel), Zozezen (the closest
+    # attention and experts: a sink, a gate per head, groups) and Qwen3 at the same width
+    "capped-small": dict(parunex=_parunex(2048, (16, 4, 128, 128), (16, 128, 128, 16), 6144, 16, 4, 4, 2, 1024, 32000),
+                         bafavik=_bafavik(2048, (16, 4, 128, 128), (16, 128, 128), (16, 4, 64, 128, 1024), (16, 16, 128, 128, 16), 6144, 32000),
+                         zozezen=_zozezen(2048, 16, 4, 128, 64, 64, 128, 8, 16, 0, 4, 1024, 2048, 32000),
+                         qwen3=dict(hidden_size=2048, intermediate_size=6144, num_attention_heads=16, num_key_value_heads=4, head_dim=128)),
+    # heads of 64 everywhere, feed-forward 10,944, 64 experts of 1,408, six per token, four of eight groups
+    "capped-lite": dict(parunex=_parunex(2048, (32, 8, 64, 64), (32, 64, 64, 32), 10944, 64, 6, 8, 4, 1408, 32000),
+                        bafavik=_bafavik(2048, (32, 8, 64, 64), (32, 64, 64), (32, 8, 64, 64, 512), (32, 32, 64, 64, 32), 10944, 32000),
+                        zozezen=_zozezen(2048, 32, 8, 64, 32, 128, 64, 4, 64, 0, 6, 1408, 2816, 32000),
+                        qwen3=dict(hidden_size=2048, intermediate_size=10944, num_attention_heads=32, num_key_value_heads=8, head_dim=64)),
 }
 
 
 def designs_workload(args) -> int:
-    """``--workload designs``: prompt and decode throughput of Vesidra, Zozezen, Kivurax, Bafavik and Venarax at sizes that resemble real models' layers, beside
+    """``--workload designs``: prompt and decode throughput of Vesidra, Zozezen, Kivurax, Bafavik, Venarax and Parunex at sizes that resemble real models' layers, beside
     the Qwen3 decoder at equal width, depth, head count and inner size; one JSON line per size and design, with each
     step's kernels (device time by kernel, from the framework profiler) so that like kernels can be set side by side."""
     import torch
@@ -761,7 +789,7 @@ def main() -> int:
                         help="fewer layers than the model has (named in the output); for quick checks only")
     parser.add_argument("--skip-points", action="store_true")
     parser.add_argument("--workload", choices=("default", "mixed", "sweep", "designs"), default="default",
-                        help="designs: Vesidra, Zozezen, Kivurax, Bafavik and Venarax beside Qwen3 at equal layer sizes (prompt and decode throughput, kernels by time)")
+                        help="designs: Vesidra, Zozezen, Kivurax, Bafavik, Venarax and Parunex beside Qwen3 at equal layer sizes (prompt and decode throughput, kernels by time)")
     parser.add_argument("--design-size", choices=sorted(DESIGN_SIZES), default=None, help="with --workload designs: one size only")
     parser.add_argument("--sweep-prompt", type=int, default=1024)
     parser.add_argument("--sweep-new", type=int, default=128)
