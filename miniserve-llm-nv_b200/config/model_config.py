@@ -1132,8 +1132,8 @@ class WavelengthRotationConfig:
 
 @dataclass(frozen=True)
 class CappedAttentionConfig:
-    """Grouped-query attention with biases on queries, keys and values, a rotation of the first ``rot.dims`` entries, scores with a
-    soft cap (``softcap``, or None), a learned sink and a gate per head.  ``v_mix``: the layer takes part in the mixing of values
+    """Grouped-query attention with biases on queries, keys and values, a rotation of the first ``rot.dims`` entries (no ``rot``: none),
+    scores with a soft cap (``softcap``, or None), a learned sink and a gate per head.  ``v_mix``: the layer takes part in the mixing of values
     along the depth (the first such layer gives its values to the others)."""
 
     heads: int
@@ -1149,9 +1149,10 @@ class CappedAttentionConfig:
     def from_dict(cls, data: Mapping[str, Any], where: str) -> "CappedAttentionConfig":
         config = cls(heads=_integer(data, "heads"), kv_heads=_integer(data, "kv_heads"), dim=_integer(data, "dim"),
                      vdim=_integer(data, "vdim"), scale=_positive(data, "scale", where),
-                     rot=WavelengthRotationConfig.from_dict(_section(data, "rot", where), where + "rot."),
+                     rot=(WavelengthRotationConfig(1.0, 0) if data.get("rot") is None
+                          else WavelengthRotationConfig.from_dict(_section(data, "rot", where), where + "rot.")),
                      softcap=None if data.get("softcap") is None else _positive(data, "softcap", where),
-                     v_mix=_boolean(data, "v_mix"))
+                     v_mix=False if data.get("v_mix") is None else _boolean(data, "v_mix"))
         if config.heads % config.kv_heads:
             raise ValueError(f"{where}heads {config.heads} is not a multiple of kv_heads {config.kv_heads}")
         if config.rot.dims > config.dim:

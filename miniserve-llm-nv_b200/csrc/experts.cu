@@ -228,9 +228,9 @@ __global__ void router_choose_kernel(const float* __restrict__ all_logits, int l
     }
     __syncwarp();
   }
-  if (lane == 0 && (normalize >= 0.f || weight_scale != 1.f)) {
-    const float factor = normalize >= 0.f ? taken + normalize : 1.f;
-    for (int k = 0; k < top; ++k) weights[(size_t)n * top + k] = weights[(size_t)n * top + k] / factor * weight_scale;
+  if (normalize >= 0.f || weight_scale != 1.f) {
+    const float factor = normalize >= 0.f ? __shfl_sync(0xffffffffu, taken, 0) + normalize : 1.f;
+    for (int k = lane; k < top; k += 32) weights[(size_t)n * top + k] = weights[(size_t)n * top + k] / factor * weight_scale;
   }
 }
 

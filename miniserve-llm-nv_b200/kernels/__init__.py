@@ -1698,7 +1698,7 @@ def linear_pair_residual(x: torch.Tensor, weight: torch.Tensor, residual: torch.
         raise KernelError(f"linear_pair_residual: weight {tuple(weight.shape)}, partials {tuple(partials.shape)} for {tiles} "
                           f"tiles of {m} rows")
     _check(library().ms_gemm_pair(_ptr(x), _ptr(weight), _ptr(x_next), _i(1), _i(3), _i(0), _i(m), _i(n), _i(k), None, _i(0),
-                                  _f(0.0), _ptr(residual), _ptr(norm_weight), _i(_code(norm_weight.dtype)), _ptr(partials), _f(0.0),
+                                  _f(0.0), _ptr(residual), _ptr(norm_weight), _i(_code(norm_weight.dtype)), _ptr(partials), _i(0), _f(0.0),
                                   _ptr(device_error_flag(x.device)), _stream()))
     return RowStats(partials, tiles, eps, per_row=True)
 

@@ -56,6 +56,10 @@ def test_configuration_reads_every_size_and_round_trips():
     del bare["layers"][0]["mlp"]["router"]["groups"], bare["layers"][0]["mixer"]["softcap"], bare["layers"][0]["mixer"]["v_mix"]
     config = ParunexConfig.from_dict(bare)
     assert (config.layers[0].mlp.group_count, config.layers[0].mixer.softcap, config.layers[0].mixer.v_mix) == (1, None, False)
+    bare["layers"][0]["mixer"].update(rot=None, v_mix=None, softcap=None)
+    bare["layers"][0]["mlp"]["router"]["groups"] = None
+    config = ParunexConfig.from_dict(bare)
+    assert (config.layers[0].mixer.rot.dims, config.layers[0].mixer.v_mix, config.layers[0].mlp.group_keep) == (0, False, 1)
 
 
 def test_the_decays_inner_size_comes_from_the_checkpoint(tmp_path):
