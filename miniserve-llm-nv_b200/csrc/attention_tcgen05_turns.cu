@@ -47,26 +47,11 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-// Two float32 operations in one instruction (packed pairs).
-__device__ __forceinline__ unsigned long long pack2(float a, float b) {
-  unsigned long long r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-  return r;
-}
-__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
-  unsigned long long r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
-}
-__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
-  unsigned long long r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-
 // A row of scores under a soft cap: v[i] = tanh(pre v[i]).  Two special-function operations a score (capped_score) would take twice
 // as long as the exponentials.  Where no score of the row exceeds half the cap, which is the usual case, the tanh's Taylor
-// series up to the thirteenth power (relative error below 2^-23 there) takes nine multiply-adds a pair instead.
+// series up to the thirteenth power (relative error about 2^-23 there) takes nine multiply-adds a pair instead.  (Giving the
+// special-function unit an eighth to a half of such a row's scores beside the series changed nothing: what counts here is how
+// many instructions the warps issue.)
 __device__ __forceinline__ void cap_row(float (&v)[BN], float twice_pre_log2) {
   float peaks[8];
 #pragma unroll
@@ -90,7 +75,7 @@ __device__ __forceinline__ void cap_row(float (&v)[BN], float twice_pre_log2) {
       s = fma2(s, y, k5);
       s = fma2(s, y, k3);
       s = fma2(mul2(x, y), s, x);
-      asm("mov.b64 {%0, %1}, %2;" : "=f"(v[i]), "=f"(v[i + 1]) : "l"(s));
+      unpack2(s, v[i], v[i + 1]);
     }
   } else {
 #pragma unroll

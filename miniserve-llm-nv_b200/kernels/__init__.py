@@ -1061,7 +1061,7 @@ def matrix_scan(mode: str, q: torch.Tensor, q_col: int, k: torch.Tensor, k_col: 
                 gates: Optional[torch.Tensor], states: torch.Tensor, state_offset: int, state_slots: torch.Tensor,
                 query_start: torch.Tensor, max_query_len: int, heads: int, kv_heads: int, dim: int, vdim: int, y: torch.Tensor,
                 q_scale: float = 1.0, bottom: Optional[torch.Tensor] = None, gate_col: int = 0,
-                channel_decay: Optional[torch.Tensor] = None, input_activation: str = "none") -> None:
+                channel_decay: Optional[torch.Tensor] = None, input_activation: str = "none", chunk: Optional[int] = None) -> None:
     """A recurrence that carries a ``dim x vdim`` matrix ``S`` per head, walked over each request's tokens from and into the
     request's state.  Queries and keys of head j are the columns ``q_col + (j // (heads / kv_heads)) dim ..`` of ``q`` (and
     ``k``), its values the columns ``v_col + j vdim ..`` of ``v`` (``q``, ``k``, ``v``: one 2-d tensor, float32 or the compute
@@ -1075,7 +1075,11 @@ def matrix_scan(mode: str, q: torch.Tensor, q_col: int, k: torch.Tensor, k_col: 
     ``"channel_delta"``: the delta form with a decay per head and key channel, ``channel_decay`` float32 ``[N, H * dim]``, acting on
     the rows of ``S``; ``gates`` is float32 ``[N, ld]`` whose columns ``gate_col .. gate_col + H`` hold the logits of beta.
     ``"channel_decay"``: ``S = diag(channel_decay) S + k v^T``, ``y = S^T q`` (a gated linear attention; ``gates`` None).  All three
-    keep ``[H, vdim, dim]``.  ``input_activation="silu"``: q, k and v pass SiLU as they are read."""
+    keep ``[H, vdim, dim]``.  ``input_activation="silu"``: q, k and v pass SiLU as they are read.
+
+    ``"channel_decay"`` of few long portions runs in chunks that need not wait for one another (a walk from zero per chunk, a join
+    of the chunks' matrices, a walk from the joined ones): ``chunk`` None lets the library choose, 0 forbids it, a number is
+    the chunk's tokens."""
     code = MATRIX_SCAN_MODES[mode]
     n = y.shape[0]
     for name, tensor in (("q", q), ("k", k), ("v", v)):
@@ -1106,6 +1110,20 @@ def matrix_scan(mode: str, q: torch.Tensor, q_col: int, k: torch.Tensor, k_col: 
     _want(query_start, "query_start", torch.int32, (n_requests + 1,))
     columns = vdim + 1 if code == 0 else vdim
     stride = _state_rows(states, state_offset, heads * columns * dim)
+    if code == 4 and chunk is None:
+        chunk = library().ms_channel_scan_chunk(_i(n_requests), _i(max_query_len), _i(heads), _i(dim), _i(vdim))
+    if chunk:
+        if code != 4 or input_activation != "none":
+            raise KernelError("matrix_scan: chunks go with the channel decay form")
+        places = n // chunk + n_requests
+        chunk_states = torch.empty((places, heads, vdim, dim), dtype=torch.float32, device=y.device)
+        chunk_decays = torch.empty((places, heads, dim), dtype=torch.float32, device=y.device)
+        _check(library().ms_channel_scan(_ptr(q), _i(q.shape[1]), _i(q_col), _ptr(k), _i(k.shape[1]), _i(k_col), _ptr(v), _i(v.shape[1]),
+                                         _i(v_col), _i(_code(q.dtype)), _f(q_scale), _ptr(channel_decay), _ptr(states), stride,
+                                         _i(state_offset), _ptr(state_slots), _ptr(query_start), _i(n_requests), _i(max_query_len),
+                                         _i(heads), _i(kv_heads), _i(dim), _i(vdim), _ptr(y), _i(chunk), _ptr(chunk_states),
+                                         _ptr(chunk_decays), _stream()))
+        return
     _check(library().ms_matrix_scan(_i(code), _ptr(q), _i(q.shape[1]), _i(q_col), _ptr(k), _i(k.shape[1]), _i(k_col), _ptr(v),
                                     _i(v.shape[1]), _i(v_col), _i(_code(q.dtype)), _f(q_scale), _ptr(gates), _ptr(states), stride,
                                     _i(state_offset), _ptr(state_slots), _ptr(query_start), _i(n_requests), _i(max_query_len),

@@ -577,7 +577,7 @@ def decay_gates(logits, a_log, dt_bias, gates):
 
 
 def matrix_scan(mode, q, q_col, k, k_col, v, v_col, gates, states, state_offset, state_slots, query_start, max_query_len, heads,
-                kv_heads, dim, vdim, y, q_scale=1.0, bottom=None, gate_col=0, channel_decay=None, input_activation="none"):
+                kv_heads, dim, vdim, y, q_scale=1.0, bottom=None, gate_col=0, channel_decay=None, input_activation="none", chunk=None):
     per = heads // kv_heads
 
     def act(x):

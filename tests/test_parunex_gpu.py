@@ -117,6 +117,54 @@ def test_matrix_scan_with_channel_decays(dtype, heads, dim, vdim):
     assert at == lengths and torch.allclose(pieces, y, atol=2e-5, rtol=2e-5) and torch.allclose(again, states, atol=2e-5, rtol=2e-5)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads,dim,vdim", [(3, 20, 12), (5, 7, 9), (4, 64, 32), (16, 128, 128), (2, 200, 40)])
+@pytest.mark.parametrize("lengths,chunk", [([40, 0, 1, 150], 16), ([33, 32, 31, 64, 65], 32), ([1, 1, 200, 1, 7], 48), ([130], 1), ([5, 2], 100)])
+def test_matrix_scan_in_chunks(dtype, heads, dim, vdim, lengths, chunk):
+    """Portions of one chunk, of several with a short last one and of exact multiples, beside single tokens and nothing at all, from
+    states that are not zero, against the plain walk; what lies around the states' rows stays as it was."""
+    from miniserve_b200 import kernels
+
+    n, slots = sum(lengths), list(range(len(lengths)))[::-1]
+    offset = 4
+    proj = rand((n, heads * (2 * dim + vdim)), dtype, 1, 0.7)
+    cols = (0, heads * dim, 2 * heads * dim)
+    decays = torch.sigmoid(rand((n, heads * dim), torch.float32, 2, 2.0) + 2.0)
+    decays[:, ::5], decays[:, 3::7] = 1.0 - 1e-4, 1e-6
+    states = rand((len(lengths) + 1, offset + heads * dim * vdim + 3), torch.float32, 3)
+    start = cpu(states)
+    y, want = torch.zeros((n, heads, vdim), device="cuda"), torch.zeros((n, heads, vdim), dtype=F64)
+    starts = torch.tensor([sum(lengths[:i]) for i in range(len(lengths) + 1)], dtype=torch.int32)
+    want_states = cpu(states).double()
+    plain_ops.matrix_scan("channel_decay", cpu(proj), cols[0], cpu(proj), cols[1], cpu(proj), cols[2], None, want_states, offset, torch.tensor(slots),
+                          starts, max(lengths), heads, heads, dim, vdim, want, q_scale=dim ** -0.5, channel_decay=cpu(decays))
+    kernels.matrix_scan("channel_decay", proj, cols[0], proj, cols[1], proj, cols[2], None, states, offset, ints(slots), starts.cuda(), max(lengths),
+                        heads, heads, dim, vdim, y, q_scale=dim ** -0.5, channel_decay=decays, chunk=chunk)
+    assert close(y, want) and torch.allclose(states.cpu().double(), want_states, atol=2e-5, rtol=2e-5)
+    assert torch.equal(states.cpu()[:, :offset], start[:, :offset]) and torch.equal(states.cpu()[:, -3:], start[:, -3:])
+    assert torch.equal(states.cpu()[-1], start[-1])
+
+
+def test_long_portions_are_scanned_in_chunks():
+    """What the library chooses: chunks for few long portions, none for many, for short ones and for keys of more than 256 entries."""
+    from miniserve_b200 import kernels
+
+    choose = kernels.library().ms_channel_scan_chunk
+    assert 64 <= choose(1, 2048, 16, 128, 128) <= 512 and choose(1, 100, 16, 128, 128) == 0 and choose(64, 512, 16, 128, 128) == 0
+    assert choose(1, 2048, 16, 300, 128) == 0
+    n, heads, dim, vdim = 700, 2, 24, 40
+    proj, decays = rand((n, heads * (2 * dim + vdim)), torch.bfloat16, 1), torch.sigmoid(rand((n, heads * dim), torch.float32, 2) + 3.0)
+    results = []
+    for chunk in (0, None):
+        states, y = torch.zeros((1, heads * dim * vdim), device="cuda"), torch.empty((n, heads, vdim), device="cuda")
+        kernels.matrix_scan("channel_decay", proj, 0, proj, heads * dim, proj, 2 * heads * dim, None, states, 0, ints([0]), ints([0, n]), n, heads,
+                            heads, dim, vdim, y, channel_decay=decays, chunk=chunk)
+        results.append((y, states))
+    assert choose(1, n, heads, dim, vdim) > 0
+    for a, b in zip(*results):
+        assert torch.allclose(a, b, atol=1e-4, rtol=1e-5) and float(a.abs().max()) > 1.0
+
+
 @pytest.mark.parametrize("rank,rows,tau,n", [(1, 12, 1.0, 1), (5, 60, 16.0, 9), (16, 300, 4.0, 70), (64, 2048, 16.0, 33)])
 def test_decays_to_a_power(rank, rows, tau, n):
     from miniserve_b200 import kernels
