@@ -60,8 +60,8 @@ __device__ __forceinline__ void load_pairs(const T* row, int sub, unsigned long 
 
 template <typename T> struct alignas(sizeof(T) * kColumns) Values { T v[kColumns]; };
 
-// LANES = 2^SHIFT (LPC above) covers the key channels.  LOCAL: the first launch (nothing is read out).  `wide`: rows of keys, queries, values and decays lie on 16-byte boundaries and hold
-// whole 16-byte pieces.
+// 2^SHIFT lanes (LPC above) cover the key channels.  LOCAL: the first launch (nothing is read out).  `wide`: rows of keys, queries,
+// values and decays lie on 16-byte boundaries and hold whole 16-byte pieces.
 template <typename T, int SHIFT, bool LOCAL>
 __global__ void __launch_bounds__(kThreads, 2)
 walk_kernel(const T* __restrict__ q, int q_ld, int q_col, const T* __restrict__ k, int k_ld, int k_col, const T* __restrict__ v, int v_ld,
